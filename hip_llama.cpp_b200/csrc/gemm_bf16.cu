@@ -17,7 +17,9 @@
 //   warp 2   TMEM allocation
 //   warps 4-7  epilogue: thread = weight row (TMEM lane), 16 columns per tcgen05.ld, optional column scale, coalesced
 //            stores (a warp writes 32 consecutive rows of one column); split-K partials to out + z * zstride
-// Up to three matrices with the same K are stacked in one launch (wq|wk|wv, w1|w3).
+// Up to three matrices with the same K are stacked in one launch (wq|wk|wv, w1|w3); or up to BF_MAX_MATS row ranges of one matrix, each
+// with activation rows of its own (BfArgs::stacked): an item's TMA coordinates start at its matrix's first weight and activation row,
+// rows of a neighbouring range that a ragged tile brings along are not stored.
 #include <stdlib.h>
 
 #include "gemm_tc.h"
@@ -29,7 +31,8 @@ constexpr int BF_THREADS = 256;
 constexpr int BF_BK = 64;             // bf16 values per k-block: 128 bytes
 
 struct BfP {
-  int M[3]; int tiles[3]; int out_off[3];
+  int M[BF_MAX_MATS]; int tiles[BF_MAX_MATS]; int out_off[BF_MAX_MATS]; int w_row[BF_MAX_MATS]; int x_row[BF_MAX_MATS];
+  int n_mats, stacked;
   int K, N, ny, kblocks_total, kblocks_per_split;
   float* out; long long ldo; long long zstride;
   const float* colscale;
@@ -86,8 +89,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap mw0, const __grid_constant_
   int* abort_flag = reinterpret_cast<int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int tiles01 = p.tiles[0] + p.tiles[1];
-  struct Item { int mat, row0, n0, kb0, nkb; };
+  struct Item { int mat, row0, n0, kb0, nkb, wrow, xrow; };
   auto item_of = [&](int it) -> Item {
     Item w;
     const int z = it % p.splits;
@@ -95,8 +97,10 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap mw0, const __grid_constant_
     int tile = t / p.ny;
     w.n0 = (t - tile * p.ny) * NT;
     w.mat = 0;
-    if (tile >= p.tiles[0]) { w.mat = 1; if (tile >= tiles01) { w.mat = 2; tile -= tiles01; } else tile -= p.tiles[0]; }
+    while (w.mat + 1 < p.n_mats && tile >= p.tiles[w.mat]) { tile -= p.tiles[w.mat]; w.mat++; }
     w.row0 = tile * (SWIGLU ? TC_BM : TC_BM * MT);
+    w.wrow = p.w_row[w.mat] + w.row0;   // where the tile lies in its tensor maps
+    w.xrow = p.x_row[w.mat] + w.n0;
     w.kb0 = z * p.kblocks_per_split;
     w.nkb = p.kblocks_total - w.kb0;
     if (w.nkb > p.kblocks_per_split) w.nkb = p.kblocks_per_split;
@@ -142,17 +146,17 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap mw0, const __grid_constant_
       };
       for (int it = blockIdx.x; it < p.n_items && ok; it += gridDim.x) {
         const Item w = item_of(it);
-        const CUtensorMap* mw = (w.mat == 0) ? &mw0 : (w.mat == 1 ? &mw1 : &mw2);
+        const CUtensorMap* mw = (w.mat == 0 || p.stacked) ? &mw0 : (w.mat == 1 ? &mw1 : &mw2);
         int i = 0;
         if (first) {
           // weights never depend on the previous kernel: the first ring goes out before the dependency wait (the bytes may
           // land before the matching expect_tx -- the phase cannot complete until that arrival)
           const int pre = w.nkb < S::NST ? w.nkb : S::NST;
-          for (; i < pre; i++) load_w(smem + i * S::STAGE, mw, (w.kb0 + i) * BF_BK, w.row0, &full[i]);
+          for (; i < pre; i++) load_w(smem + i * S::STAGE, mw, (w.kb0 + i) * BF_BK, w.wrow, &full[i]);
           pdl_wait();
           for (int j = 0; j < pre; j++) {
             tc_mbar_expect_tx(&full[j], S::STAGE);
-            tc_tma_2d(smem + j * S::STAGE + S::W_BYTES, &mx, (w.kb0 + j) * BF_BK, w.n0, &full[j]);
+            tc_tma_2d(smem + j * S::STAGE + S::W_BYTES, &mx, (w.kb0 + j) * BF_BK, w.xrow, &full[j]);
           }
           first = false;
         }
@@ -160,8 +164,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap mw0, const __grid_constant_
           const int g = gb + i, s = g % S::NST;
           if (g >= S::NST && !tc_mbar_wait(&empty[s], ((g / S::NST) & 1u) ^ 1u, abort_flag)) { ok = false; break; }
           tc_mbar_expect_tx(&full[s], S::STAGE);
-          load_w(smem + s * S::STAGE, mw, (w.kb0 + i) * BF_BK, w.row0, &full[s]);
-          tc_tma_2d(smem + s * S::STAGE + S::W_BYTES, &mx, (w.kb0 + i) * BF_BK, w.n0, &full[s]);
+          load_w(smem + s * S::STAGE, mw, (w.kb0 + i) * BF_BK, w.wrow, &full[s]);
+          tc_tma_2d(smem + s * S::STAGE + S::W_BYTES, &mx, (w.kb0 + i) * BF_BK, w.xrow, &full[s]);
         }
         gb += w.nkb;
       }
@@ -306,10 +310,12 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap mw0, const __grid_constant_
 
 // ------------------------------------------------------------------ host side ----
 bool gemm_bf16_ok(const BfArgs& a) {
-  if (a.K % 8 || a.ldx % 8 || a.K < BF_BK || a.N < 1 || a.n_mats < 1 || a.n_mats > 3 || !a.X || !a.out) return false;
+  if (a.K % 8 || a.ldx % 8 || a.K < BF_BK || a.N < 1 || a.n_mats < 1 || a.n_mats > (a.stacked ? BF_MAX_MATS : 3) || !a.X || !a.out) return false;
   if (reinterpret_cast<uintptr_t>(a.X) & 15u) return false;
-  for (int i = 0; i < a.n_mats; i++)
-    if (!a.W[i] || (reinterpret_cast<uintptr_t>(a.W[i]) & 15u) || a.M[i] < 1) return false;
+  for (int i = 0; i < a.n_mats; i++) {
+    const uint16_t* w = a.W[a.stacked ? 0 : i];
+    if (!w || (reinterpret_cast<uintptr_t>(w) & 15u) || a.M[i] < 1) return false;
+  }
   return true;
 }
 
@@ -346,7 +352,22 @@ int gemm_bf16_launch(cudaStream_t st, const BfArgs& a, bool pdl) {
   CUtensorMap mw[3], mx;
   BfP p = {};
   int tiles = 0;
-  for (int i = 0; i < 3; i++) {
+  p.n_mats = a.n_mats; p.stacked = a.stacked;
+  int x_rows = a.N;
+  if (a.stacked) {
+    if (swiglu) return THA_STATUS_NOT_SUPPORTED;
+    int w_rows = 0;
+    for (int i = 0; i < a.n_mats; i++) {
+      p.M[i] = a.M[i]; p.tiles[i] = ceil_div(a.M[i], TC_BM * MT); p.out_off[i] = a.out_off[i];
+      p.w_row[i] = a.w_row[i]; p.x_row[i] = a.x_row[i];
+      w_rows = max(w_rows, a.w_row[i] + a.M[i]);
+      x_rows = max(x_rows, a.x_row[i] + a.N);
+      tiles += p.tiles[i];
+    }
+    THA_TRY_RC(tc_map(a.W[0], w_rows, a.K, a.K, TC_BM * MT, &mw[0], 2));
+    mw[1] = mw[2] = mw[0];
+  }
+  for (int i = 0; i < 3 && !a.stacked; i++) {
     if (i < a.n_mats) {
       THA_TRY_RC(tc_map(a.W[i], a.M[i], a.K, a.K, TC_BM * MT, &mw[i], 2));
       p.M[i] = a.M[i]; p.tiles[i] = ceil_div(a.M[i], TC_BM * MT); p.out_off[i] = a.out_off[i];
@@ -356,7 +377,7 @@ int gemm_bf16_launch(cudaStream_t st, const BfArgs& a, bool pdl) {
     tiles += p.tiles[i];
   }
   if (swiglu) { tiles = p.tiles[0]; p.tiles[1] = 0; p.swiglu_out = a.swiglu_out; p.ld_swiglu = a.ld_swiglu; }   // an item = a pair of tiles
-  THA_TRY_RC(tc_map(a.X, a.N, a.K, a.ldx, NT, &mx, 2));
+  THA_TRY_RC(tc_map(a.X, x_rows, a.K, a.ldx, NT, &mx, 2));
   p.K = a.K; p.N = a.N;
   p.kblocks_total = ceil_div(a.K, BF_BK);
   const int splits = a.splits < 1 ? 1 : a.splits;

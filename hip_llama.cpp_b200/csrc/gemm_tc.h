@@ -39,8 +39,9 @@ int gemm_q8i_pick_nt(int N, int gs);
 int gemm_q8i_launch(cudaStream_t st, const Q8iArgs& a, bool pdl);
 
 // bf16 weights x bf16 activations (gemm_bf16.cu): both operands straight from TMA-written shared memory
+constexpr int BF_MAX_MATS = 8;
 struct BfArgs {
-  int n_mats; const uint16_t* W[3]; int M[3]; int out_off[3];
+  int n_mats; const uint16_t* W[3]; int M[BF_MAX_MATS]; int out_off[BF_MAX_MATS];
   int K;
   const uint16_t* X; int N; long long ldx;       // activations [N, ldx] bf16
   float* out; long long ldo; long long zstride; int splits;
@@ -49,6 +50,9 @@ struct BfArgs {
   // of w1 AND the same 128 rows of w3; its read-out writes silu(w1 x) * (w3 x), rounded to bf16, to swiglu_out[n * ld_swiglu + row]
   // (the input of the w2 matmul) and `out` is not written at all.
   uint16_t* swiglu_out; long long ld_swiglu;
+  // stacked: up to BF_MAX_MATS matrices that are row ranges of ONE matrix W[0], each with activation rows of its own: matrix i =
+  // rows w_row[i] .. + M[i] of W[0], its activations rows x_row[i] .. + N of X
+  int stacked; int w_row[BF_MAX_MATS]; int x_row[BF_MAX_MATS];
 };
 bool gemm_bf16_swiglu_ok(const BfArgs& a);   // the launch can take the SwiGLU read-out
 bool gemm_bf16_ok(const BfArgs& a);

@@ -19,9 +19,9 @@
 namespace tha {
 
 template <typename T>
-__global__ void hyb_add_norm_kernel(float* __restrict__ x, const float* __restrict__ left, float c_left, const float* __restrict__ right,
+__global__ void hyb_add_norm_kernel(float* __restrict__ x, const float* __restrict__ left, const float* __restrict__ left_b, float c_left, const float* __restrict__ right,
                                     float c_right, const float* __restrict__ embed_out, const float* __restrict__ vec, tha_norm_t n,
-                                    int has_norm, float eps, T* __restrict__ out, int width) {
+                                    int has_norm, float eps, T* __restrict__ out, long long ldo, int width) {
   __shared__ float red[33];
   const int r = blockIdx.x;
   float* xr = x + (size_t)r * width;
@@ -29,7 +29,7 @@ __global__ void hyb_add_norm_kernel(float* __restrict__ x, const float* __restri
   for (int i = threadIdx.x; i < width; i += blockDim.x) {
     float v = xr[i];
     if (left) {
-      float y = c_left * left[(size_t)r * width + i];
+      float y = c_left * (left[(size_t)r * width + i] + (left_b ? left_b[i] : 0.f));
       if (right) y = fmaf(c_right, right[(size_t)r * width + i], y);
       v += y;
     }
@@ -46,17 +46,17 @@ __global__ void hyb_add_norm_kernel(float* __restrict__ x, const float* __restri
     for (int i = threadIdx.x; i < width; i += blockDim.x) { const float d = xr[i] - mean; ss = fmaf(d, d, ss); }
     ss = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)width + eps);
-    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * width + i, fmaf((xr[i] - mean) * inv, n.w[i], n.b ? n.b[i] : 0.f));
+    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * ldo + i, fmaf((xr[i] - mean) * inv, n.w[i], n.b ? n.b[i] : 0.f));
   } else if (n.kind == THA_NORM_RMS) {
     float ss = 0.f;
     for (int i = threadIdx.x; i < width; i += blockDim.x) ss = fmaf(xr[i], xr[i], ss);
     ss = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)width + eps);
-    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * width + i, xr[i] * inv * (n.w_offset + n.w[i]));
+    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * ldo + i, xr[i] * inv * (n.w_offset + n.w[i]));
   } else if (n.kind == THA_NORM_DYT) {
-    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * width + i, fmaf(tanhf(n.alpha * xr[i]), n.w[i], n.b ? n.b[i] : 0.f));
+    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * ldo + i, fmaf(tanhf(n.alpha * xr[i]), n.w[i], n.b ? n.b[i] : 0.f));
   } else {   // THA_NORM_COPY
-    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * width + i, xr[i]);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * ldo + i, xr[i]);
   }
 }
 
@@ -76,9 +76,9 @@ __global__ void hyb_side_gate_kernel(T* __restrict__ out, const float* __restric
 // projection), the tap; then what comes ahead of the NEXT layer run -- the embedding output and the pass vector (nullable) --
 // and its first norm, so that the next layer starts at its stacked product.
 template <typename T>
-__global__ void hyb_block_finish_kernel(float* __restrict__ x, const float* __restrict__ ff, const float* __restrict__ y, float m,
-                                        const float* __restrict__ w, float eps, float* __restrict__ tap, const float* __restrict__ embed_out,
-                                        const float* __restrict__ vec, tha_norm_t n, int has_norm, T* __restrict__ out, int width) {
+__global__ void hyb_block_finish_kernel(float* __restrict__ x, const float* __restrict__ ff, const float* __restrict__ ff_b, const float* __restrict__ y,
+                                        float m, const float* __restrict__ w, float eps, float* __restrict__ tap, const float* __restrict__ embed_out,
+                                        const float* __restrict__ vec, tha_norm_t n, int has_norm, T* __restrict__ out, long long ldo, int width) {
   __shared__ float red[33];
   const int r = blockIdx.x;
   float* xr = x + (size_t)r * width;
@@ -92,7 +92,7 @@ __global__ void hyb_block_finish_kernel(float* __restrict__ x, const float* __re
   float sum = 0.f;
   for (int i = threadIdx.x; i < width; i += blockDim.x) {
     float v = xr[i];
-    if (ff) v = fmaf(m, ff[(size_t)r * width + i], v);
+    if (ff) v = fmaf(m, ff[(size_t)r * width + i] + (ff_b ? ff_b[i] : 0.f), v);
     if (y) v = fmaf(y[(size_t)r * width + i] * inv, w[i], v);
     if (tap) tap[(size_t)r * width + i] = v;
     if (embed_out) v += embed_out[(size_t)r * width + i];
@@ -108,17 +108,17 @@ __global__ void hyb_block_finish_kernel(float* __restrict__ x, const float* __re
     for (int i = threadIdx.x; i < width; i += blockDim.x) { const float d = xr[i] - mean; ss = fmaf(d, d, ss); }
     ss = block_sum(ss, red);
     const float iv = 1.0f / sqrtf(ss / (float)width + eps);
-    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * width + i, fmaf((xr[i] - mean) * iv, n.w[i], n.b ? n.b[i] : 0.f));
+    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * ldo + i, fmaf((xr[i] - mean) * iv, n.w[i], n.b ? n.b[i] : 0.f));
   } else if (n.kind == THA_NORM_RMS) {
     float ss = 0.f;
     for (int i = threadIdx.x; i < width; i += blockDim.x) ss = fmaf(xr[i], xr[i], ss);
     ss = block_sum(ss, red);
     const float iv = 1.0f / sqrtf(ss / (float)width + eps);
-    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * width + i, xr[i] * iv * (n.w_offset + n.w[i]));
+    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * ldo + i, xr[i] * iv * (n.w_offset + n.w[i]));
   } else if (n.kind == THA_NORM_DYT) {
-    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * width + i, fmaf(tanhf(n.alpha * xr[i]), n.w[i], n.b ? n.b[i] : 0.f));
+    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * ldo + i, fmaf(tanhf(n.alpha * xr[i]), n.w[i], n.b ? n.b[i] : 0.f));
   } else {
-    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * width + i, xr[i]);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) hyb_store(out + (size_t)r * ldo + i, xr[i]);
   }
 }
 
@@ -133,18 +133,19 @@ static int block_threads(int width) {
   return t;
 }
 
-extern "C" int tha_hyb_add_norm(void* stream, int dtype, float* x, const float* left, float c_left, const float* right, float c_right,
-                                const float* embed_out, const float* vec, const tha_norm_t* n, float eps, void* out, int n_rows, int width) {
+extern "C" int tha_hyb_add_norm(void* stream, int dtype, float* x, const float* left, const float* left_b, float c_left, const float* right,
+                                float c_right, const float* embed_out, const float* vec, const tha_norm_t* n, float eps, void* out, long long ldo,
+                                int n_rows, int width) {
   if (n_rows < 1) return THA_STATUS_SUCCESS;
   if (!x || (n && (!out || (!n->w && n->kind != THA_NORM_COPY)))) return THA_STATUS_INVALID_ARG;
   const tha_norm_t none = {};
   const int nt = block_threads(width);
   if (dtype == THA_DT_BF16)
-    THA_CUDA_OK(launch(hyb_add_norm_kernel<bf16>, dim3(n_rows), dim3(nt), 0, (cudaStream_t)stream, false, x, left, c_left, right, c_right, embed_out, vec,
-                       n ? *n : none, n ? 1 : 0, eps, (bf16*)out, width));
+    THA_CUDA_OK(launch(hyb_add_norm_kernel<bf16>, dim3(n_rows), dim3(nt), 0, (cudaStream_t)stream, false, x, left, left_b, c_left, right, c_right, embed_out, vec,
+                       n ? *n : none, n ? 1 : 0, eps, (bf16*)out, ldo > 0 ? ldo : (long long)width, width));
   else
-    THA_CUDA_OK(launch(hyb_add_norm_kernel<float>, dim3(n_rows), dim3(nt), 0, (cudaStream_t)stream, false, x, left, c_left, right, c_right, embed_out,
-                       vec, n ? *n : none, n ? 1 : 0, eps, (float*)out, width));
+    THA_CUDA_OK(launch(hyb_add_norm_kernel<float>, dim3(n_rows), dim3(nt), 0, (cudaStream_t)stream, false, x, left, left_b, c_left, right, c_right, embed_out,
+                       vec, n ? *n : none, n ? 1 : 0, eps, (float*)out, ldo > 0 ? ldo : (long long)width, width));
   return THA_STATUS_SUCCESS;
 }
 
@@ -162,18 +163,18 @@ extern "C" int tha_hyb_side_gate(void* stream, int dtype, void* out, const float
   return THA_STATUS_SUCCESS;
 }
 
-extern "C" int tha_hyb_block_finish(void* stream, int dtype, float* x, const float* ff, const float* y, float m, const float* y_norm, float eps,
-                                    float* tap, const float* embed_out, const float* vec, const tha_norm_t* next_norm, void* out, int n_rows,
-                                    int width) {
+extern "C" int tha_hyb_block_finish(void* stream, int dtype, float* x, const float* ff, const float* ff_b, const float* y, float m, const float* y_norm,
+                                    float eps, float* tap, const float* embed_out, const float* vec, const tha_norm_t* next_norm, void* out,
+                                    long long ldo, int n_rows, int width) {
   if (n_rows < 1) return THA_STATUS_SUCCESS;
   if (!x || (y && !y_norm) || (next_norm && (!out || (!next_norm->w && next_norm->kind != THA_NORM_COPY)))) return THA_STATUS_INVALID_ARG;
   const tha_norm_t none = {};
   const int nt = block_threads(width);
   if (dtype == THA_DT_BF16)
-    THA_CUDA_OK(launch(hyb_block_finish_kernel<bf16>, dim3(n_rows), dim3(nt), 0, (cudaStream_t)stream, false, x, ff, y, m, y_norm, eps, tap, embed_out,
-                       vec, next_norm ? *next_norm : none, next_norm ? 1 : 0, (bf16*)out, width));
+    THA_CUDA_OK(launch(hyb_block_finish_kernel<bf16>, dim3(n_rows), dim3(nt), 0, (cudaStream_t)stream, false, x, ff, ff_b, y, m, y_norm, eps, tap, embed_out,
+                       vec, next_norm ? *next_norm : none, next_norm ? 1 : 0, (bf16*)out, ldo > 0 ? ldo : (long long)width, width));
   else
-    THA_CUDA_OK(launch(hyb_block_finish_kernel<float>, dim3(n_rows), dim3(nt), 0, (cudaStream_t)stream, false, x, ff, y, m, y_norm, eps, tap, embed_out,
-                       vec, next_norm ? *next_norm : none, next_norm ? 1 : 0, (float*)out, width));
+    THA_CUDA_OK(launch(hyb_block_finish_kernel<float>, dim3(n_rows), dim3(nt), 0, (cudaStream_t)stream, false, x, ff, ff_b, y, m, y_norm, eps, tap, embed_out,
+                       vec, next_norm ? *next_norm : none, next_norm ? 1 : 0, (float*)out, ldo > 0 ? ldo : (long long)width, width));
   return THA_STATUS_SUCCESS;
 }

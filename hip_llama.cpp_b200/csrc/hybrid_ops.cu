@@ -285,6 +285,21 @@ __global__ void hyb_attn_prepare_kernel(tha_attn_t a, tha_rows_t rows, tha_kv_t 
   const int n_k = a.kv_shared ? 0 : a.kv_heads, n_v = a.kv_shared ? 0 : a.kv_heads / (a.v_share > 1 ? a.v_share : 1);
   // queries grow with the logarithm of their position, in steps of q_temp_every positions
   const float q_mult = a.q_temp_every > 0 ? 1.0f + a.q_temp_coef * logf((float)((t + 1) / a.q_temp_every + 1)) : 1.0f;
+  // row norms: one mean over all heads' channels, taken by the whole block before the heads are dealt to its warps
+  float row_q = 1.0f, row_k = 1.0f;
+  if (a.q_norm || a.k_norm) {
+    __shared__ float red[33];
+    if (a.q_norm) {
+      float ss = 0.f;
+      for (int i = threadIdx.x; i < a.heads * a.dim; i += blockDim.x) { const float v = pr[a.o_q + i]; ss = fmaf(v, v, ss); }
+      row_q = 1.0f / sqrtf(block_sum(ss, red) / (float)(a.heads * a.dim) + a.eps);
+    }
+    if (a.k_norm && n_k) {
+      float ss = 0.f;
+      for (int i = threadIdx.x; i < a.kv_heads * a.dim; i += blockDim.x) { const float v = pr[a.o_k + i]; ss = fmaf(v, v, ss); }
+      row_k = 1.0f / sqrtf(block_sum(ss, red) / (float)(a.kv_heads * a.dim) + a.eps);
+    }
+  }
   for (int h = warp; h < a.heads + n_k + n_v; h += nwarps) {
     if (h >= a.heads + n_k) {   // a value head: plain copy
       const int g = h - a.heads - n_k;
@@ -297,13 +312,15 @@ __global__ void hyb_attn_prepare_kernel(tha_attn_t a, tha_rows_t rows, tha_kv_t 
     // the first rot_dims entries rotated (pairs by the layout), the rest passed through
     const float* cr = cos_t + (size_t)r * half;
     const float* sr = sin_t + (size_t)r * half;
+    const float* wn = is_q ? a.q_norm : a.k_norm;   // per-channel weights sit inside the rotation, the row's factor outside
+    if (wn) wn += is_q ? h * a.dim : (h - a.heads) * a.dim;
     float ss = 0.f;
     if (a.unit_rms) {
-      for (int d = lane; d < a.dim; d += 32) { const float v = hyb_rotated(src, d, rot_dims, a.rot_layout, cr, sr); ss = fmaf(v, v, ss); }
+      for (int d = lane; d < a.dim; d += 32) { const float v = hyb_rotated(src, d, rot_dims, a.rot_layout, cr, sr, wn); ss = fmaf(v, v, ss); }
       ss = warp_sum(ss);
     }
-    const float inv = (a.unit_rms ? 1.0f / sqrtf(ss / (float)a.dim + a.eps) : 1.0f) * (is_q ? q_mult : 1.0f);
-    for (int d = lane; d < a.dim; d += 32) dst[d] = hyb_rotated(src, d, rot_dims, a.rot_layout, cr, sr) * inv;
+    const float inv = (a.unit_rms ? 1.0f / sqrtf(ss / (float)a.dim + a.eps) : 1.0f) * (is_q ? q_mult * row_q : row_k);
+    for (int d = lane; d < a.dim; d += 32) dst[d] = hyb_rotated(src, d, rot_dims, a.rot_layout, cr, sr, wn) * inv;
   }
 }
 
@@ -447,7 +464,8 @@ __global__ void __launch_bounds__(128) hyb_attn_kernel(tha_attn_t a, tha_rows_t 
 #pragma unroll
     for (int rr = 0; rr < 4; rr++) {
       const bool vis = my_ok[rr] && hyb_attn_sees(a, t, my_pos[rr], my_first[rr]);
-      const float sv = vis ? sc[rr] * a.scale * my_scale[rr] : -INFINITY;
+      float sv = vis ? sc[rr] * a.scale * my_scale[rr] : -INFINITY;
+      if (a.softcap > 0.f && vis) sv = hyb_softcap(sv, a.softcap);
       const float m_new = fmaxf(m_run[rr], warp_max(sv));
       float p = 0.f, corr = 1.f;
       if (m_new > -INFINITY) {
@@ -545,7 +563,13 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<const uint32_t*>(&v);
 }
 
-template <bool EXACT>
+// cap * tanh(s / cap) as cap * (1 - 2 / (1 + e^(2 s / cap))): its absolute error is a few 1e-7 of the cap, the size of an fp32 score's
+// own rounding at the cap
+__device__ __forceinline__ float attn_softcap_fast(float s, float cap, float two_over_cap) {
+  return cap - __fdividef(2.0f * cap, 1.0f + __expf(s * two_over_cap));
+}
+
+template <bool EXACT, bool CAP>
 __global__ void __launch_bounds__(128, 3) hyb_attn_mma_kernel(tha_attn_t a, tha_rows_t rows, tha_kv_t kv, const float* __restrict__ q,
                                                            __nv_bfloat16* __restrict__ out, int AG, int AP, int splits,
                                                            float* __restrict__ partial, const float* __restrict__ gate, long long ldg) {
@@ -600,6 +624,7 @@ __global__ void __launch_bounds__(128, 3) hyb_attn_mma_kernel(tha_attn_t a, tha_
       qf[ks][2 + x] = ok ? pack_bf16(qr[16 * ks + 8 + lc], qr[16 * ks + 8 + lc + 1]) : 0u;
     }
   }
+  const float two_over_cap = CAP ? 2.0f / a.softcap : 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   float oacc[AM_MAXD / 8][4];
 #pragma unroll
@@ -713,7 +738,9 @@ __global__ void __launch_bounds__(128, 3) hyb_attn_mma_kernel(tha_attn_t a, tha_
         for (int y = 0; y < 2; y++) {
           const int t = kt + 8 * j + lc + y;
           const bool vis = row_ok[x] && hyb_attn_sees(a, t, row_pos[x], row_first[x]);
-          const float sv = vis ? sacc[j][2 * x + y] * a.scale * row_scale[x] : -INFINITY;
+          float sv = sacc[j][2 * x + y] * a.scale * row_scale[x];
+          if (CAP) sv = attn_softcap_fast(sv, a.softcap, two_over_cap);
+          if (!vis) sv = -INFINITY;
           sacc[j][2 * x + y] = sv;
           mx = fmaxf(mx, sv);
         }
@@ -1135,7 +1162,7 @@ __global__ void hyb_head_gate_kernel(T* __restrict__ out, const float* __restric
   for (int e = lane; e < E; e += 32) {
     const float z = gate ? gate[(size_t)r * ldg + h * E + e] : 0.f;
     const float g = !gate ? 1.0f : gate_act == THA_GATE_SILU ? z * hyb_sigmoid(z) : hyb_sigmoid(z);
-    const float v = do_norm ? o[e] * inv * norm[norm_per_head ? h * E + e : e] : o[e];
+    const float v = do_norm ? o[e] * inv * (norm ? norm[norm_per_head ? h * E + e : e] : 1.0f) : o[e];
     hyb_store(out + (size_t)r * heads * E + (size_t)h * E + e, v * g);
   }
 }
@@ -1148,8 +1175,8 @@ __global__ void hyb_head_gate_kernel(T* __restrict__ out, const float* __restric
 constexpr int CONV_MAX_TAPS = 8;
 template <typename T, int V>
 __global__ void hyb_conv_kernel(tha_rows_t rows, tha_state_store_t st, long long conv_state_off, const float* __restrict__ proj,
-                                long long ldp, int col0, int channels, int taps, const float* __restrict__ w, int act, int add_input,
-                                T* __restrict__ out) {
+                                long long ldp, int col0, int channels, int taps, const float* __restrict__ w, const float* __restrict__ bias,
+                                int act, int add_input, T* __restrict__ out) {
   const int c = V * (blockIdx.x * blockDim.x + threadIdx.x);
   if (c >= channels) return;
   float wr[CONV_MAX_TAPS][V];
@@ -1157,6 +1184,9 @@ __global__ void hyb_conv_kernel(tha_rows_t rows, tha_state_store_t st, long long
   for (int j = 0; j < CONV_MAX_TAPS; j++)
 #pragma unroll
     for (int v = 0; v < V; v++) wr[j][v] = j < taps ? w[(size_t)(c + v) * taps + j] : 0.f;
+  float bv[V];
+#pragma unroll
+  for (int v = 0; v < V; v++) bv[v] = bias ? bias[c + v] : 0.f;
   for (int r = blockIdx.y; r < rows.n_rows; r += gridDim.y) {
     const int s = rows.row_seq[r], first = rows.seq_first[s];
     const float* tail = st.base + (size_t)rows.seq_slot[s] * st.slot_floats + conv_state_off + (size_t)c * (taps - 1);
@@ -1170,6 +1200,8 @@ __global__ void hyb_conv_kernel(tha_rows_t rows, tha_state_store_t st, long long
       if (rr >= first) {
         if (V == 4) { const float4 t = *reinterpret_cast<const float4*>(proj + (size_t)rr * ldp + col0 + c); x[0] = t.x; x[1] = t.y; x[2] = t.z; x[3] = t.w; }
         else x[0] = proj[(size_t)rr * ldp + col0 + c];
+#pragma unroll
+        for (int v = 0; v < V; v++) x[v] += bv[v];
       } else {
 #pragma unroll
         for (int v = 0; v < V; v++) x[v] = tail[(size_t)v * (taps - 1) + (taps - 1) - (first - rr)];
@@ -1198,34 +1230,36 @@ __global__ void hyb_conv_kernel(tha_rows_t rows, tha_state_store_t st, long long
 // any number of taps, a channel per thread
 template <typename T>
 __global__ void hyb_conv_long_kernel(tha_rows_t rows, tha_state_store_t st, long long conv_state_off, const float* __restrict__ proj,
-                                     long long ldp, int col0, int channels, int taps, const float* __restrict__ w, int act, int add_input,
-                                     T* __restrict__ out) {
+                                     long long ldp, int col0, int channels, int taps, const float* __restrict__ w,
+                                     const float* __restrict__ bias, int act, int add_input, T* __restrict__ out) {
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= channels) return;
+  const float bv = bias ? bias[c] : 0.f;
   for (int r = blockIdx.y; r < rows.n_rows; r += gridDim.y) {
     const int s = rows.row_seq[r], first = rows.seq_first[s];
     const float* tail = st.base + (size_t)rows.seq_slot[s] * st.slot_floats + conv_state_off + (size_t)c * (taps - 1);
     float acc = 0.f;
     for (int j = 0; j < taps; j++) {
       const int rr = r - (taps - 1 - j);
-      const float x = rr >= first ? proj[(size_t)rr * ldp + col0 + c] : tail[(taps - 1) - (first - rr)];
+      const float x = rr >= first ? proj[(size_t)rr * ldp + col0 + c] + bv : tail[(taps - 1) - (first - rr)];
       acc = fmaf(w[(size_t)c * taps + j], x, acc);
     }
     if (act == 1) acc = acc / (1.0f + expf(-acc));
-    if (add_input) acc += proj[(size_t)r * ldp + col0 + c];
+    if (add_input) acc += proj[(size_t)r * ldp + col0 + c] + bv;
     hyb_store(out + (size_t)r * channels + c, acc);
   }
 }
 // after the convolution: tail[i] <- the input (taps-1-i) tokens before the end of what the sequence has seen now
 __global__ void hyb_conv_tail_kernel(tha_rows_t rows, tha_state_store_t st, long long conv_state_off, const float* __restrict__ proj,
-                                     long long ldp, int col0, int channels, int taps) {
+                                     long long ldp, int col0, int channels, int taps, const float* __restrict__ bias) {
   const int c = blockIdx.x * blockDim.x + threadIdx.x, s = blockIdx.y;
   if (c >= channels) return;
+  const float bv = bias ? bias[c] : 0.f;
   const int first = rows.seq_first[s], n = rows.seq_first[s + 1] - first;
   float* tail = st.base + (size_t)rows.seq_slot[s] * st.slot_floats + conv_state_off + (size_t)c * (taps - 1);
   for (int i = 0; i < taps - 1; i++) {           // ascending: tail[i + n] is read before it is overwritten
     const int back = (taps - 1) - i;             // this entry is the input `back` tokens before the end
-    tail[i] = back <= n ? proj[(size_t)(first + n - back) * ldp + col0 + c] : tail[i + n];
+    tail[i] = back <= n ? proj[(size_t)(first + n - back) * ldp + col0 + c] + bv : tail[i + n];
   }
 }
 
@@ -1585,7 +1619,6 @@ extern "C" int tha_hyb_linear_heads(void* stream, int dtype, float* C, long long
 extern "C" int tha_hyb_head_gate(void* stream, int dtype, void* out, const float* o_raw, int n_rows, int heads, int E, int do_norm,
                                  float eps, const float* norm, int norm_per_head, const float* gate, long long ldg, int gate_act) {
   if (n_rows < 1) return THA_STATUS_SUCCESS;
-  if (do_norm && !norm) return THA_STATUS_INVALID_ARG;
   const dim3 grid(ceil_div(n_rows * heads, 4));
   if (dtype == THA_DT_BF16)
     THA_CUDA_OK(launch(hyb_head_gate_kernel<bf16>, grid, dim3(128), 0, (cudaStream_t)stream, false, (bf16*)out, o_raw, n_rows, heads, E, eps, norm,
@@ -1630,6 +1663,30 @@ extern "C" int tha_hyb_linear(void* stream, int dtype, float* C, long long ldc, 
   return THA_STATUS_SUCCESS;
 }
 
+extern "C" int tha_hyb_linear_groups(void* stream, int dtype, float* C, long long ldc, const void* A, const void* W, int M, int K, int n_groups,
+                                     const int* group_n_host) {
+  if (M < 1 || n_groups < 1) return THA_STATUS_SUCCESS;
+  if (K < 1 || !C || !A || !W || !group_n_host || n_groups > BF_MAX_MATS) return THA_STATUS_INVALID_ARG;
+  if (dtype == THA_DT_BF16 && hyb_tc_linear()) {
+    // one launch of the tcgen05 matmul: its work items carry their group's first weight row and first input row
+    BfArgs b = {};
+    b.n_mats = n_groups; b.stacked = 1; b.W[0] = (const uint16_t*)W; b.K = K;
+    b.X = (const uint16_t*)A; b.N = M; b.ldx = K;
+    b.out = C; b.ldo = ldc; b.splits = 1;
+    for (int g = 0, at = 0; g < n_groups; at += group_n_host[g], g++) {
+      b.M[g] = group_n_host[g]; b.out_off[g] = at; b.w_row[g] = at; b.x_row[g] = g * M;
+    }
+    if (gemm_bf16_ok(b)) return gemm_bf16_launch((cudaStream_t)stream, b, false);
+  }
+  const size_t es = dtype == THA_DT_BF16 ? 2 : 4;
+  for (int g = 0, at = 0; g < n_groups; at += group_n_host[g], g++) {
+    const int st = tha_hyb_linear(stream, dtype, C + at, ldc, (const char*)A + (size_t)g * M * K * es, K, 0, nullptr, (const char*)W + (size_t)at * K * es,
+                                  0, M, group_n_host[g], K, nullptr, 0);
+    if (st != THA_STATUS_SUCCESS) return st;
+  }
+  return THA_STATUS_SUCCESS;
+}
+
 extern "C" int tha_hyb_rotary_table(void* stream, const tha_rotary_t* rot, const int* pos, int n_rows, float* cos_out, float* sin_out) {
   const int half = rot->dims / 2;
   if (n_rows < 1 || half < 1) return THA_STATUS_SUCCESS;
@@ -1642,7 +1699,7 @@ extern "C" int tha_hyb_attn_prepare(void* stream, const tha_attn_t* a, const tha
                                     long long ldp, const float* cos_t, const float* sin_t, int rot_dims, float* q_out) {
   if (rows->n_rows < 1) return THA_STATUS_SUCCESS;
   if (a->heads % a->kv_heads || rot_dims > a->dim || (rot_dims & 1) || a->kv_heads * a->dim > kv->kv_dim ||
-      a->kv_heads / (a->v_share > 1 ? a->v_share : 1) * a->vdim > kv->kv_dim)
+      a->kv_heads / (a->v_share > 1 ? a->v_share : 1) * a->vdim > kv->kv_dim || (a->v_is_k && a->vdim != a->dim))
     return THA_STATUS_INVALID_ARG;
   const int nt = pick_threads(32 * (a->heads + 2 * a->kv_heads));
   THA_CUDA_OK(launch(hyb_attn_prepare_kernel, dim3(rows->n_rows), dim3(nt), 0, (cudaStream_t)stream, false, *a, *rows, *kv, proj, ldp, cos_t,
@@ -1682,7 +1739,7 @@ extern "C" int tha_hyb_attn_gated(void* stream, int dtype, const tha_attn_t* a, 
   // bf16 with heads the tensor-core form covers: 64 pairs per block; else 16 pairs on the fp32 cores
   const bool tc = dtype == THA_DT_BF16 && hyb_tc_linear() && hyb_tc_attn() && a->dim % 16 == 0 && a->vdim % 8 == 0 && a->dim <= AM_MAXD && a->vdim <= AM_MAXD &&
                   (a->heads * a->vdim) % 2 == 0;
-  const bool wide = !tc && !gate && !a->head_scale && !a->out_f32 && a->v_share <= 1 && dtype == THA_DT_BF16 && hyb_tc_linear() && hyb_tc_attn() && hyb_attn_wide_ok(a);
+  const bool wide = !tc && !gate && !a->head_scale && a->softcap <= 0.f && !a->out_f32 && a->v_share <= 1 && dtype == THA_DT_BF16 && hyb_tc_linear() && hyb_tc_attn() && hyb_attn_wide_ok(a);
   const int pairs = wide ? hyb_attn_wide_pairs(a, rows) : tc ? AM_PAIRS : ATT_PAIRS;
   const int AG = gsize < pairs ? gsize : pairs, AP = pairs / AG;
   const size_t smem = tc ? sizeof(__nv_bfloat16) * ((size_t)ATT_KEYS * (a->dim + 8) + (size_t)ATT_KEYS * (a->vdim + 8))
@@ -1709,10 +1766,12 @@ extern "C" int tha_hyb_attn_gated(void* stream, int dtype, const tha_attn_t* a, 
       const int st = hyb_attn_wide_launch(s, a, rows, kv, q, (bf16*)out, grid, pairs, AG, AP, splits, split_scratch);
       if (st != THA_STATUS_SUCCESS) return st;
     } else if (tc) {
-      if (a->fp32_scores)
-        THA_CUDA_OK(launch(hyb_attn_mma_kernel<true>, grid, dim3(128), smem, s, false, *a, *rows, *kv, q, (bf16*)out, AG, AP, splits, split_scratch, gate, ldg));
+      if (a->softcap > 0.f)
+        THA_CUDA_OK(launch(hyb_attn_mma_kernel<true, true>, grid, dim3(128), smem, s, false, *a, *rows, *kv, q, (bf16*)out, AG, AP, splits, split_scratch, gate, ldg));
+      else if (a->fp32_scores)
+        THA_CUDA_OK(launch(hyb_attn_mma_kernel<true, false>, grid, dim3(128), smem, s, false, *a, *rows, *kv, q, (bf16*)out, AG, AP, splits, split_scratch, gate, ldg));
       else
-        THA_CUDA_OK(launch(hyb_attn_mma_kernel<false>, grid, dim3(128), smem, s, false, *a, *rows, *kv, q, (bf16*)out, AG, AP, splits, split_scratch, gate, ldg));
+        THA_CUDA_OK(launch(hyb_attn_mma_kernel<false, false>, grid, dim3(128), smem, s, false, *a, *rows, *kv, q, (bf16*)out, AG, AP, splits, split_scratch, gate, ldg));
     } else {
       if (a->vdim <= 256) {
         if (smem > 48 * 1024) THA_CUDA_OK(cudaFuncSetAttribute(hyb_attn_kernel<bf16, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
@@ -1785,8 +1844,8 @@ extern "C" int tha_hyb_mem_scan(void* stream, int dtype, const tha_mem_t* m, con
 }
 
 extern "C" int tha_hyb_conv(void* stream, int dtype, const tha_rows_t* rows, const tha_state_store_t* st, long long conv_state_off,
-                            const float* proj, long long ldp, int col0, int channels, int taps, const float* w, int act, int add_input,
-                            int out_f32, void* out) {
+                            const float* proj, long long ldp, int col0, int channels, int taps, const float* w, const float* bias, int act,
+                            int add_input, int out_f32, void* out) {
   if (rows->n_rows < 1 || channels < 1) return THA_STATUS_SUCCESS;
   if (taps < 1) return THA_STATUS_INVALID_ARG;
   cudaStream_t s = (cudaStream_t)stream;
@@ -1797,9 +1856,9 @@ extern "C" int tha_hyb_conv(void* stream, int dtype, const tha_rows_t* rows, con
     /* about eight blocks per SM: a block walks several rows with its taps in registers */                                               \
     const int gy = min(rows->n_rows, max(1, 148 * 8 / gx));                                                                               \
     const dim3 grid(gx, gy);                                                                                                              \
-    if (f32) THA_CUDA_OK(launch(KF, grid, dim3(128), 0, s, false, *rows, *st, conv_state_off, proj, ldp, col0, channels, taps, w, act, add_input, \
+    if (f32) THA_CUDA_OK(launch(KF, grid, dim3(128), 0, s, false, *rows, *st, conv_state_off, proj, ldp, col0, channels, taps, w, bias, act, add_input, \
                                 (float*)out));                                                                                            \
-    else THA_CUDA_OK(launch(KB, grid, dim3(128), 0, s, false, *rows, *st, conv_state_off, proj, ldp, col0, channels, taps, w, act, add_input,     \
+    else THA_CUDA_OK(launch(KB, grid, dim3(128), 0, s, false, *rows, *st, conv_state_off, proj, ldp, col0, channels, taps, w, bias, act, add_input,     \
                             (bf16*)out));                                                                                                 \
   } while (0)
   if (taps > CONV_MAX_TAPS) CONV_GO(hyb_conv_long_kernel<float>, hyb_conv_long_kernel<bf16>, 1);
@@ -1810,17 +1869,17 @@ extern "C" int tha_hyb_conv(void* stream, int dtype, const tha_rows_t* rows, con
   return THA_STATUS_SUCCESS;
 }
 extern "C" int tha_hyb_conv_tail(void* stream, const tha_rows_t* rows, const tha_state_store_t* st, long long conv_state_off,
-                                 const float* proj, long long ldp, int col0, int channels, int taps) {
+                                 const float* proj, long long ldp, int col0, int channels, int taps, const float* bias) {
   if (rows->n_rows < 1 || channels < 1 || taps <= 1) return THA_STATUS_SUCCESS;
   THA_CUDA_OK(launch(hyb_conv_tail_kernel, dim3(ceil_div(channels, 128), rows->n_seqs), dim3(128), 0, (cudaStream_t)stream, false, *rows, *st,
-                     conv_state_off, proj, ldp, col0, channels, taps));
+                     conv_state_off, proj, ldp, col0, channels, taps, bias));
   return THA_STATUS_SUCCESS;
 }
 extern "C" int tha_hyb_conv_silu(void* stream, const tha_rows_t* rows, const tha_state_store_t* st, long long conv_state_off,
                                  const float* proj, long long ldp, int col0, int channels, int taps, const float* w, float* out) {
-  const int status = tha_hyb_conv(stream, THA_DT_F32, rows, st, conv_state_off, proj, ldp, col0, channels, taps, w, 1, 0, 1, out);
+  const int status = tha_hyb_conv(stream, THA_DT_F32, rows, st, conv_state_off, proj, ldp, col0, channels, taps, w, nullptr, 1, 0, 1, out);
   if (status != THA_STATUS_SUCCESS) return status;
-  return tha_hyb_conv_tail(stream, rows, st, conv_state_off, proj, ldp, col0, channels, taps);
+  return tha_hyb_conv_tail(stream, rows, st, conv_state_off, proj, ldp, col0, channels, taps, nullptr);
 }
 
 extern "C" int tha_hyb_delta_scan(void* stream, int dtype, const tha_delta_t* d, const tha_rows_t* rows, const tha_state_store_t* st,

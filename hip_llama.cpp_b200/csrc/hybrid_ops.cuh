@@ -18,16 +18,23 @@ __device__ __forceinline__ float hyb_softplus(float z) { return fmaxf(z, 0.f) + 
 
 // Element d of a vector whose first rot_dims entries are rotated by the row's angles (c, s: cos and sin of its rot_dims / 2
 // pairs): the pair (first, second) becomes (first c - second s, second c + first s).  THA_ROT_INTERLEAVED pairs (2i, 2i + 1),
-// THA_ROT_HALVES pairs (i, i + rot_dims / 2); entries from rot_dims on pass unchanged.
-__device__ __forceinline__ float hyb_rotated(const float* src, int d, int rot_dims, int layout, const float* c, const float* s) {
-  if (d >= rot_dims) return src[d];
+// THA_ROT_HALVES pairs (i, i + rot_dims / 2); entries from rot_dims on pass unchanged.  w (nullable): per-entry weights applied first.
+__device__ __forceinline__ float hyb_rotated(const float* src, int d, int rot_dims, int layout, const float* c, const float* s,
+                                             const float* w = nullptr) {
+  if (d >= rot_dims) return w ? src[d] * w[d] : src[d];
   const int half = rot_dims >> 1;
   const bool first = layout == THA_ROT_HALVES ? d < half : !(d & 1);
   const int i = layout == THA_ROT_HALVES ? (first ? d : d - half) : d >> 1;
   const int partner = layout == THA_ROT_HALVES ? (first ? d + half : d - half) : d ^ 1;
-  const float x = src[d], y = src[partner];
+  const float x = w ? src[d] * w[d] : src[d], y = w ? src[partner] * w[partner] : src[partner];
   return first ? x * c[i] - y * s[i] : x * c[i] + y * s[i];
 }
+
+// The scanned memories (hybrid_gla.cu): forms of the recurrence and the launch they share.  dec [n_rows, heads * dim]: decays per key
+// channel (not SCAN_HEAD_DECAY); aux: [heads] decays (SCAN_HEAD_DECAY) or [heads * dim] bonus (SCAN_BONUS).
+enum { SCAN_CHANNEL_DECAY = 0, SCAN_HEAD_DECAY = 1, SCAN_BONUS = 2 };
+int hyb_scan_launch(cudaStream_t s, int form, const tha_gla_t* g, const tha_rows_t* rows, const tha_state_store_t* st, const float* proj, long long ldp,
+                    const float* dec, const float* aux, float* o_raw, float qscale);
 
 // first float of the cache row of (slot, position t) in cache layer `layer` of a pool
 __device__ __forceinline__ size_t hyb_kv_row(const tha_kv_t& kv, int slot, int t, int layer) {

@@ -15,10 +15,12 @@
 namespace tha {
 
 // x = embed[token] * scale (+ the learned vector of the row's position when the model has a position table); x0, when given,
-// keeps a copy of it for the layers that add the embedding output again
+// keeps a copy of it for the layers that add the embedding output again; join [rows, 2 width], when given, gets both halves of the
+// joining map's input [x; embedding output] (the second half stays for the whole step)
 template <typename T>
 __global__ void hyb_embed_kernel(float* __restrict__ x, const T* __restrict__ embed, const int* __restrict__ token, int width,
-                                 const T* __restrict__ pos_embed, const int* __restrict__ pos, float scale, float* __restrict__ x0) {
+                                 const T* __restrict__ pos_embed, const int* __restrict__ pos, float scale, float* __restrict__ x0,
+                                 T* __restrict__ join) {
   const int r = blockIdx.x;
   const T* e = embed + (size_t)token[r] * width;
   const T* p = pos_embed ? pos_embed + (size_t)pos[r] * width : nullptr;
@@ -26,6 +28,7 @@ __global__ void hyb_embed_kernel(float* __restrict__ x, const T* __restrict__ em
     const float v = hyb_load(e + i) * scale + (p ? hyb_load(p + i) : 0.f);
     x[(size_t)r * width + i] = v;
     if (x0) x0[(size_t)r * width + i] = v;
+    if (join) { hyb_store(join + (size_t)r * 2 * width + i, v); hyb_store(join + (size_t)r * 2 * width + width + i, v); }
   }
 }
 
@@ -98,6 +101,7 @@ struct StepBuffers {
   float *proj2, *qfull, *x0, *sgate;
   float *xs, *hf, *att;   // the residual streams [rows, n, width]; a normed input before its convolution; fp32 attention maps
   void* sg;
+  void *join, *mix;        // the joining map's input [rows, 2 width]; the token-shifted inputs [5][rows, width]
   void *h, *h2, *cq, *qplain, *abuf, *mbuf, *y, *sy, *hn, *hg;
   int *expert_id, *group_off, *sorted_row, *inv;
   float* cos_t[64]; float* sin_t[64];
@@ -113,10 +117,11 @@ static long long hyb_expert_rows() {
   return (v && *v) ? atoll(v) : 1024;
 }
 
-// channels of an attention layer's short convolution: its projected q | k | v columns (q alone when it reads another layer's rows)
+// channels of an attention layer's short convolution: its projected q | k | v columns (q alone when it reads another layer's rows,
+// q | k when the values are the keys)
 static size_t hyb_attn_conv_channels(const tha_attn_t& a) {
   size_t c = (size_t)a.heads * a.dim;
-  if (!a.kv_shared) c += (size_t)a.kv_heads * a.dim + (size_t)(a.kv_heads / (a.v_share > 1 ? a.v_share : 1)) * a.vdim;
+  if (!a.kv_shared) c += (size_t)a.kv_heads * a.dim + (a.v_is_k ? 0 : (size_t)(a.kv_heads / (a.v_share > 1 ? a.v_share : 1)) * a.vdim);
   return c;
 }
 
@@ -125,7 +130,7 @@ static size_t carve(const tha_hyb_model_t* m, int R, int n_want, char* base, Ste
   const size_t W = m->width, es = m->dtype == THA_DT_BF16 ? 2 : 4;
   size_t n_in = 0, qd = 0, av = 0, mv = 0, cc = 0, dd = 0, dg = 0, gu = 0, ff = 0, sff = 0, top = 0, ne = 0;
   size_t n_in2 = 0, qr = 0, qf = 0, qp = 0;
-  bool norm2 = false, keep_embed = false;
+  bool norm2 = false, keep_embed = false, join = false, shift = false;
   size_t sd = 0, n_str = 0, hfw = 0, attf = 0;
   for (int i = 0; i < m->n_layers; i++) {
     const tha_hyb_layer_t& L = m->layers[i];
@@ -133,6 +138,7 @@ static size_t carve(const tha_hyb_model_t* m, int R, int n_want, char* base, Ste
     if (L.block == THA_BLOCK_STREAMS) n_str = (size_t)(m->n_streams > 0 ? m->n_streams : 1);
     if (L.in_conv_taps > 0) hfw = W;
     if (L.pre_add_embed) keep_embed = true;
+    if (L.w_join) join = true;
     sd = max(sd, (size_t)L.side.dim);
     if (L.mixer == THA_MIX_ATTN || L.mixer == THA_MIX_ATTN_GDELTA) {
       qd = max(qd, (size_t)L.attn.heads * L.attn.dim);
@@ -144,6 +150,13 @@ static size_t carve(const tha_hyb_model_t* m, int R, int n_want, char* base, Ste
       dd = max(dd, (size_t)L.hgrn.heads * L.hgrn.dim);
       mv = max(mv, (size_t)L.hgrn.heads * L.hgrn.vdim);
     }
+    if (L.mixer == THA_MIX_WKV) {
+      shift = true;
+      hfw = W;
+      dd = max(dd, (size_t)L.wkv.heads * L.wkv.dim);
+      mv = max(mv, (size_t)L.wkv.heads * L.wkv.dim);
+    }
+    if (L.mixer == THA_MIX_RETENTION) mv = max(mv, (size_t)L.retention.heads * L.retention.vdim);
     if (L.mixer == THA_MIX_ATTN_GDELTA) {
       dd = max(dd, (size_t)L.gdelta.heads * L.gdelta.dim);
       mv = max(mv, (size_t)L.gdelta.heads * L.gdelta.dim);
@@ -185,6 +198,8 @@ static size_t carve(const tha_hyb_model_t* m, int R, int n_want, char* base, Ste
   if (!keep_embed) b->x0 = nullptr;
   b->xs = c.take<float>(R * n_str * W);
   b->hf = c.take<float>(R * hfw);
+  b->join = join ? c.take<char>(2 * R * W * es) : nullptr;
+  b->mix = c.take<char>(shift ? 5 * R * W * es : 0);
   b->att = c.take<float>(R * attf);
   b->h = c.take<char>(R * W * es);
   b->proj = c.take<float>(R * n_in);
@@ -304,13 +319,18 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
   const float embed_scale = m->embed_scale != 0.f ? m->embed_scale : 1.0f;
   if (dt == THA_DT_BF16)
     THA_CUDA_OK(launch(hyb_embed_kernel<bf16>, dim3(R), dim3(128), 0, s, false, b.x, (const bf16*)m->embed, rows->token, W, (const bf16*)m->pos_embed,
-                       rows->pos, embed_scale, b.x0));
+                       rows->pos, embed_scale, b.x0, (bf16*)b.join));
   else
     THA_CUDA_OK(launch(hyb_embed_kernel<float>, dim3(R), dim3(128), 0, s, false, b.x, (const float*)m->embed, rows->token, W,
-                       (const float*)m->pos_embed, rows->pos, embed_scale, b.x0));
+                       (const float*)m->pos_embed, rows->pos, embed_scale, b.x0, (float*)b.join));
   for (int i = 0; i < m->n_rot; i++) HYB_OK(tha_hyb_rotary_table(stream, &m->rot[i], rows->pos, R, b.cos_t[i], b.sin_t[i]));
 
-  bool h_ready = false;   // the previous block's last pass already left this layer's first norm in b.h
+  bool h_ready = false;   // the previous block's last pass already left this layer's first norm in b.h (b.hf: see norm_out)
+  bool join_ready = b.join != nullptr;   // the first half of b.join holds the current x
+  // where a sequential layer's first norm goes, and in which format: a token-shifted mixer mixes it in fp32 first
+  const tha_norm_t copy_x = {THA_NORM_COPY};
+  auto norm_out = [&](const tha_hyb_layer_t& X) -> void* { return X.mixer == THA_MIX_WKV ? (void*)b.hf : b.h; };
+  auto norm_dt = [&](const tha_hyb_layer_t& X) { return X.mixer == THA_MIX_WKV ? THA_DT_F32 : dt; };
   for (int li = 0; li < m->n_layers; li++) {
     const tha_hyb_layer_t& L = m->layers[li];
     const long long ldp = L.n_in;
@@ -327,15 +347,34 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
                                nullptr, &L.streams1, &L.norm1, m->eps, conv, conv ? (void*)b.hf : b.h, R, W));
       h_ready = false;
       if (conv) {
-        HYB_OK(tha_hyb_conv(stream, dt, rows, st, L.in_conv_state_off, b.hf, W, 0, W, L.in_conv_taps, L.in_conv_w, 0, 1, 0, b.h));
-        HYB_OK(tha_hyb_conv_tail(stream, rows, st, L.in_conv_state_off, b.hf, W, 0, W, L.in_conv_taps));
+        HYB_OK(tha_hyb_conv(stream, dt, rows, st, L.in_conv_state_off, b.hf, W, 0, W, L.in_conv_taps, L.in_conv_w, nullptr, 0, 1, 0, b.h));
+        HYB_OK(tha_hyb_conv_tail(stream, rows, st, L.in_conv_state_off, b.hf, W, 0, W, L.in_conv_taps, nullptr));
       }
     } else if (seq && h_ready) h_ready = false;
-    else if (seq && (L.pre_add_embed || L.pre_vec))   // a pass's re-entry addends and the mixer's norm in one pass over x
-      HYB_OK(tha_hyb_add_norm(stream, dt, b.x, nullptr, 0.f, nullptr, 0.f, L.pre_add_embed ? b.x0 : nullptr, L.pre_vec, &L.norm1, m->eps, b.h, R, W));
+    else if (seq) {
+      if (L.w_join) {   // x <- W_join [x; embedding output]
+        if (!join_ready)
+          HYB_OK(tha_hyb_add_norm(stream, dt, b.x, nullptr, nullptr, 0.f, nullptr, 0.f, nullptr, nullptr, &copy_x, m->eps, b.join, 2 * W, R, W));
+        HYB_OK(tha_hyb_linear(stream, dt, b.x, W, b.join, 2 * W, 0, nullptr, L.w_join, 0, R, W, 2 * W, nullptr, 0));
+      }
+      if (L.pre_add_embed || L.pre_vec)   // a pass's re-entry addends and the mixer's norm in one pass over x
+        HYB_OK(tha_hyb_add_norm(stream, norm_dt(L), b.x, nullptr, nullptr, 0.f, nullptr, 0.f, L.pre_add_embed ? b.x0 : nullptr, L.pre_vec, &L.norm1,
+                                m->eps, norm_out(L), 0, R, W));
+      else
+        HYB_OK(tha_hyb_norm(stream, norm_dt(L), norm_out(L), b.x, &L.norm1, m->eps, R, W, nullptr));
+    }
     else if (two_norms) HYB_OK(tha_hyb_norm_pair(stream, dt, b.h, b.h2, b.x, &L.norm1, &L.norm2, m->eps, R, W));
     else HYB_OK(tha_hyb_norm(stream, dt, b.h, b.x, &L.norm1, m->eps, R, W, nullptr));
-    HYB_OK(tha_hyb_linear(stream, dt, b.proj, ldp, b.h, W, 0, nullptr, L.w_in, 0, R, L.n_in, W, nullptr, 0));
+    join_ready = false;
+    if (L.mixer == THA_MIX_WKV) {
+      // five mixes of every row with its predecessor, each the input of a product of its own: one grouped launch
+      const int hd = L.wkv.heads * L.wkv.dim;
+      const int group_n[5] = {hd, hd, hd, hd, L.wkv.rank};
+      HYB_OK(tha_hyb_token_shift(stream, dt, rows, st, L.wkv.shift_state_off, b.hf, W, L.wkv.mu, 5, b.mix));
+      HYB_OK(tha_hyb_linear_groups(stream, dt, b.proj, ldp, b.mix, L.w_in, R, W, 5, group_n));
+    } else {
+      HYB_OK(tha_hyb_linear(stream, dt, b.proj, ldp, b.h, W, 0, nullptr, L.w_in, 0, R, L.n_in, W, nullptr, 0));
+    }
     const float* right = nullptr;
     if (L.mixer == THA_MIX_ATTN || L.mixer == THA_MIX_ATTN_GDELTA) {
       const tha_attn_t& a = L.attn;
@@ -346,9 +385,9 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
       long long ldq = ldp;
       if (a.conv_taps > 0) {
         const int C = (int)hyb_attn_conv_channels(a);
-        HYB_OK(tha_hyb_conv(stream, dt, rows, st, a.conv_state_off, b.proj, ldp, a.o_q, C, a.conv_taps, a.conv_w, 0, 0, 1, b.conv));
-        HYB_OK(tha_hyb_conv_tail(stream, rows, st, a.conv_state_off, b.proj, ldp, a.o_q, C, a.conv_taps));
-        ap.o_q = 0; ap.o_k = a.heads * a.dim; ap.o_v = ap.o_k + a.kv_heads * a.dim;
+        HYB_OK(tha_hyb_conv(stream, dt, rows, st, a.conv_state_off, b.proj, ldp, a.o_q, C, a.conv_taps, a.conv_w, a.conv_b, 0, 0, 1, b.conv));
+        HYB_OK(tha_hyb_conv_tail(stream, rows, st, a.conv_state_off, b.proj, ldp, a.o_q, C, a.conv_taps, a.conv_b));
+        ap.o_q = 0; ap.o_k = a.heads * a.dim; ap.o_v = a.v_is_k ? ap.o_k : ap.o_k + a.kv_heads * a.dim;
         pq = b.conv; ldq = C;
       }
       HYB_OK(tha_hyb_attn_prepare(stream, &ap, rows, kv, pq, ldq, a.rot >= 0 ? b.cos_t[a.rot] : nullptr,
@@ -396,6 +435,15 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
     } else if (L.mixer == THA_MIX_HGRN) {
       const tha_hgrn_t& g = L.hgrn;
       HYB_OK(tha_hyb_hgrn_scan(stream, dt, &g, rows, st, b.proj, ldp, b.dt_raw, b.oraw, b.mbuf));
+      HYB_OK(tha_hyb_linear(stream, dt, b.left, W, b.mbuf, g.heads * g.vdim, 0, nullptr, g.w_o, 0, R, W, g.heads * g.vdim, nullptr, 0));
+    } else if (L.mixer == THA_MIX_WKV) {
+      const tha_wkv_t& g = L.wkv;
+      HYB_OK(tha_hyb_wkv_scan(stream, dt, &g, rows, st, b.proj, ldp, b.dt_raw, b.oraw, b.mbuf));
+      HYB_OK(tha_hyb_linear(stream, dt, b.left, W, b.mbuf, g.heads * g.dim, 0, nullptr, g.w_o, 0, R, W, g.heads * g.dim, nullptr, 0));
+    } else if (L.mixer == THA_MIX_RETENTION) {
+      const tha_retention_t& g = L.retention;
+      HYB_OK(tha_hyb_retention_scan(stream, dt, &g, rows, st, b.proj, ldp, g.rot >= 0 ? b.cos_t[g.rot] : nullptr, g.rot >= 0 ? b.sin_t[g.rot] : nullptr,
+                                    g.rot >= 0 ? m->rot[g.rot].dims : 0, b.oraw, b.mbuf));
       HYB_OK(tha_hyb_linear(stream, dt, b.left, W, b.mbuf, g.heads * g.vdim, 0, nullptr, g.w_o, 0, R, W, g.heads * g.vdim, nullptr, 0));
     } else if (L.mixer == THA_MIX_LATENT) {
       const tha_latent_t& a = L.latent;
@@ -470,15 +518,21 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
       const float m_res = L.res_mult;
       const float cl = L.mixer == THA_MIX_ATTN_GDELTA ? m_res * L.mix_left : m_res, cr = m_res * L.mix_right;
       const float* ffo = nullptr;
+      const float* ffb = nullptr;
+      const bool has_attn = L.mixer == THA_MIX_ATTN || L.mixer == THA_MIX_ATTN_GDELTA;
+      const float* left_b = has_attn ? L.attn.b_o : nullptr;
       if (L.has_ff == THA_FF_DENSE) {
         const tha_dense_ff_t& d = L.dense;
-        HYB_OK(tha_hyb_add_norm(stream, dt, b.x, b.left, cl, right, cr, nullptr, nullptr, &L.norm2, m->eps, b.h2, R, W));
+        HYB_OK(tha_hyb_add_norm(stream, dt, b.x, b.left, left_b, cl, right, cr, nullptr, nullptr, &L.norm2, m->eps, b.h2, 0, R, W));
         HYB_OK(tha_hyb_linear(stream, dt, b.proj2, L.n_in2, b.h2, W, 0, nullptr, L.w_in2, 0, R, L.n_in2, W, nullptr, 0));
         HYB_OK(tha_hyb_ff_act(stream, dt, d.act, b.sy, b.proj2, L.n_in2, d.o_gate, d.o_up, R, d.ff, d.act_p, d.act_q));
         HYB_OK(tha_hyb_linear(stream, dt, b.sdown, W, b.sy, d.ff, 0, nullptr, d.w_down, 0, R, W, d.ff, nullptr, 0));
         ffo = b.sdown;
+      } else if (L.has_ff == THA_FF_NONE && !right) {
+        ffo = b.left;   // the mixer's own residual add joins the last pass over x
+        ffb = left_b;
       } else if (L.has_ff == THA_FF_NONE) {
-        HYB_OK(tha_hyb_add_norm(stream, dt, b.x, b.left, cl, right, cr, nullptr, nullptr, nullptr, m->eps, nullptr, R, W));
+        HYB_OK(tha_hyb_add_norm(stream, dt, b.x, b.left, left_b, cl, right, cr, nullptr, nullptr, nullptr, m->eps, nullptr, 0, R, W));
       } else {
         return THA_STATUS_NOT_SUPPORTED;
       }
@@ -486,8 +540,7 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
       if (L.side.dim > 0) {
         // the side input reads the stream after the feed-forward: x += m * ff and x in the products' number format, the gate
         // product, its activation times the token's table entries, the projection
-        const tha_norm_t copy = {THA_NORM_COPY};
-        HYB_OK(tha_hyb_add_norm(stream, dt, b.x, ffo, m_res, nullptr, 0.f, nullptr, nullptr, &copy, m->eps, b.h, R, W));
+        HYB_OK(tha_hyb_add_norm(stream, dt, b.x, ffo, ffb, m_res, nullptr, 0.f, nullptr, nullptr, &copy_x, m->eps, b.h, 0, R, W));
         ffo = nullptr;
         HYB_OK(tha_hyb_linear(stream, dt, b.sgate, L.side.dim, b.h, W, 0, nullptr, L.side.w_gate, 0, R, L.side.dim, W, nullptr, 0));
         HYB_OK(tha_hyb_side_gate(stream, dt, b.sg, b.sgate, L.side.dim, &L.side, m->side_table, m->side_cols, rows->token, R));
@@ -496,9 +549,15 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
       }
       // the last pass over x: the remaining residual adds, the tap, and what comes ahead of the next layer run
       const tha_hyb_layer_t* next = li + 1 < m->n_layers && m->layers[li + 1].block == THA_BLOCK_SEQUENTIAL ? &m->layers[li + 1] : nullptr;
-      HYB_OK(tha_hyb_block_finish(stream, dt, b.x, ffo, y, m_res, L.side.norm, m->eps, taps ? taps + (size_t)li * R * W : (float*)nullptr,
+      float* tap = taps ? taps + (size_t)li * R * W : (float*)nullptr;
+      if (next && next->w_join) {   // the next run starts with its joining map: x goes to the map's input instead of through a norm
+        HYB_OK(tha_hyb_block_finish(stream, dt, b.x, ffo, ffb, y, m_res, L.side.norm, m->eps, tap, nullptr, nullptr, &copy_x, b.join, 2 * W, R, W));
+        join_ready = true;
+        continue;
+      }
+      HYB_OK(tha_hyb_block_finish(stream, next ? norm_dt(*next) : dt, b.x, ffo, ffb, y, m_res, L.side.norm, m->eps, tap,
                                   next && next->pre_add_embed ? b.x0 : nullptr, next ? next->pre_vec : nullptr, next ? &next->norm1 : nullptr,
-                                  next ? b.h : nullptr, R, W));
+                                  next ? norm_out(*next) : nullptr, 0, R, W));
       h_ready = next != nullptr;
       continue;
     }

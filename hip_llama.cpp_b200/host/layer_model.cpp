@@ -18,6 +18,7 @@ void register_timerax();   // host/arch_timerax.cpp
 void register_numizen();   // host/arch_numizen.cpp
 void register_bozovik();   // host/arch_bozovik.cpp
 void register_mozetar();   // host/arch_mozetar.cpp
+void register_logulix();   // host/arch_logulix.cpp
 
 // ---- registry -----------------------------------------------------------------------------------------------------
 static std::vector<ArchitectureEntry>& registry() {
@@ -32,6 +33,7 @@ static void register_builtin() {
     register_numizen();
     register_bozovik();
     register_mozetar();
+    register_logulix();
   });
 }
 void register_architecture(const ArchitectureEntry& e) {
@@ -281,6 +283,10 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
           }
           mag = (float)(0.1 * log(rs.factor) + 1.0);
         }
+        if (rs.linear) {
+          if (!(rs.factor > 0.0)) throw std::runtime_error("rotary scaling: the factor must be positive");
+          for (int i = 0; i < half; i++) f[i] /= rs.factor;
+        }
         if (rs.by_wavelength) {
           if (!(rs.high > rs.low) || !(rs.factor > 0.0) || !(rs.original > 0.0)) throw std::runtime_error("rotary scaling: needs high > low, factor > 0, original > 0");
           for (int i = 0; i < half; i++) {
@@ -321,6 +327,9 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
       const int maps = a.diff ? 2 : 1;   // score maps per head: a differential head owns two query rows and two key rows
       A.heads = a.heads * maps; A.kv_heads = a.kv_heads * maps;
       const long long cq = (long long)A.heads * a.dim, ck = (long long)A.kv_heads * a.dim, cv = (long long)a.kv_heads * a.vdim;
+      if (a.v_is_k && (a.vdim != a.dim || a.diff || a.kv_from >= 0)) throw std::runtime_error("attention: values that are the keys need vdim == dim, one map per head and rows of their own");
+      if ((!a.q_norm.empty() || !a.k_norm.empty()) && a.diff) throw std::runtime_error("attention: row norms of differential projections are not served");
+      if (a.softcap < 0.f) throw std::runtime_error("attention: the score cap must be positive");
       m->separate_values_ = true;
       if (a.kv_from >= 0) {
         // the rows of an earlier layer: same head counts and rotation, nothing of its own in the cache
@@ -359,15 +368,37 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
       }
       if (a.kv_from < 0) {
         A.o_k = in.add(a.k, ck);
-        A.o_v = in.add(a.v, cv);
+        if (a.v_is_k) { A.v_is_k = 1; A.o_v = A.o_k; }
+        else A.o_v = in.add(a.v, cv);
       }
+      A.softcap = a.softcap;
+      if (!a.q_norm.empty()) A.q_norm = vec(a.q_norm, (size_t)cq);
+      if (!a.k_norm.empty() && a.kv_from < 0) A.k_norm = vec(a.k_norm, (size_t)ck);
+      if (!a.o_b.empty()) A.b_o = vec(a.o_b, W);
       A.q_temp_coef = a.q_temp_coef; A.q_temp_every = a.q_temp_every > 0 ? a.q_temp_every : 0;
+      const bool biased = !a.q_b.empty() || !a.k_b.empty();
+      if (biased && (a.diff || a.kv_from >= 0 || !a.v_is_k)) throw std::runtime_error("attention: projection biases are served where the values are the keys");
+      if (biased) {   // added ahead of the convolution
+        std::vector<float> b;
+        if (!a.q_b.empty()) file.read_f32(a.q_b, &b); else b.resize((size_t)cq, 0.f);
+        if ((long long)b.size() != cq) throw std::runtime_error("tensor '" + a.q_b + "': one bias per projected channel is expected");
+        if (!a.k_b.empty()) file.read_f32(a.k_b, &b); else b.resize((size_t)(cq + ck), 0.f);
+        if ((long long)b.size() != cq + ck) throw std::runtime_error("tensor '" + a.k_b + "': one bias per projected channel is expected");
+        A.conv_b = (const float*)m->upload(b.data(), b.size() * 4);
+        if (a.conv_taps <= 0) {   // no convolution: one tap of one, which adds the bias and nothing else
+          std::vector<float> one((size_t)(cq + ck), 1.f);
+          A.conv_taps = 1;
+          A.conv_w = (const float*)m->upload(one.data(), one.size() * 4);
+          A.conv_state_off = state;
+        }
+      }
       if (a.conv_taps > 0) {
         if (a.diff) throw std::runtime_error("attention: a short convolution behind differential projections is not served");
         std::vector<float> taps;
         file.read_f32(a.q + ".conv", &taps);
-        if (a.kv_from < 0) { file.read_f32(a.k + ".conv", &taps); file.read_f32(a.v + ".conv", &taps); }
-        const long long C = cq + (a.kv_from < 0 ? ck + cv : 0);
+        if (a.kv_from < 0) file.read_f32(a.k + ".conv", &taps);
+        if (a.kv_from < 0 && !a.v_is_k) file.read_f32(a.v + ".conv", &taps);
+        const long long C = cq + (a.kv_from < 0 ? ck + (a.v_is_k ? 0 : cv) : 0);
         if ((long long)taps.size() != C * a.conv_taps) throw std::runtime_error("attention: convolution taps do not fit [channels, " + std::to_string(a.conv_taps) + "]");
         A.conv_taps = a.conv_taps;
         A.conv_w = (const float*)m->upload(taps.data(), taps.size() * 4);
@@ -395,6 +426,13 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
       }
       return it->second + (size_t)row * W;
     };
+    std::map<std::string, const void*> joins;
+    auto join_matrix = [&](const std::string& name) -> const void* {
+      if (name.empty()) return nullptr;
+      auto it = joins.find(name);
+      if (it == joins.end()) it = joins.emplace(name, mat(name, W, 2 * W)).first;
+      return it->second;
+    };
     for (size_t li = 0; li < spec.layers.size(); li++) {
       li_now = li;
       const LayerSpec& ls = spec.layers[li];
@@ -411,8 +449,26 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
           L.hgrn.state_off = state;
           state += (long long)L.hgrn.heads * L.hgrn.dim * ((L.hgrn.vdim + 7) / 8 * 8);
         }
-        if ((L.mixer == THA_MIX_ATTN || L.mixer == THA_MIX_ATTN_GDELTA) && (L.attn.kv_shared || L.attn.conv_taps > 0))
-          throw std::runtime_error("a repeated attention layer with a short convolution or another layer's cache rows is not served");
+        L.w_join = join_matrix(ls.pre_join);
+        if ((L.mixer == THA_MIX_ATTN || L.mixer == THA_MIX_ATTN_GDELTA) && L.attn.kv_shared)
+          throw std::runtime_error("a repeated attention layer with another layer's cache rows is not served");
+        if ((L.mixer == THA_MIX_ATTN || L.mixer == THA_MIX_ATTN_GDELTA) && L.attn.conv_taps > 0) {
+          const tha_attn_t& A = L.attn;
+          const long long C = (long long)A.heads * A.dim + (long long)A.kv_heads * A.dim +
+                              (A.v_is_k ? 0 : (long long)(A.kv_heads / (A.v_share > 1 ? A.v_share : 1)) * A.vdim);
+          L.attn.conv_state_off = state;
+          state += C * (A.conv_taps - 1);
+        }
+        if (L.mixer == THA_MIX_WKV) {
+          L.wkv.state_off = state;
+          state += tha_hyb_scan_state_floats(L.wkv.heads, L.wkv.dim, L.wkv.dim);
+          L.wkv.shift_state_off = state;
+          state += W;
+        }
+        if (L.mixer == THA_MIX_RETENTION) {
+          L.retention.state_off = state;
+          state += tha_hyb_scan_state_floats(L.retention.heads, L.retention.dim, L.retention.vdim);
+        }
         if (L.mixer == THA_MIX_ATTN || L.mixer == THA_MIX_ATTN_GDELTA) {
           L.attn.cache_layer = m->n_cache_layers_++;
           if (L.mixer == THA_MIX_ATTN_GDELTA) {
@@ -442,6 +498,9 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
       L.res_mult = ls.res_mult;
       L.pre_add_embed = ls.pre_add_embed ? 1 : 0;
       if (!ls.pre_vec.empty()) L.pre_vec = pre_vector(ls.pre_vec, ls.pre_vec_row);
+      L.w_join = join_matrix(ls.pre_join);
+      if (ls.block != THA_BLOCK_SEQUENTIAL && (!ls.pre_join.empty() || !ls.attn.o_b.empty() || ls.mixer == THA_MIX_WKV))
+        throw std::runtime_error("a joining map, an output bias and token-shifted mixers are served in sequential blocks");
       if (ls.block == THA_BLOCK_SEQUENTIAL && ls.has_ff && (ls.ff_kind != THA_FF_DENSE || ls.norm2.empty()))
         throw std::runtime_error("a sequential block serves a dense feed-forward behind a second norm, or none");
       L.norm1 = norm(ls.norm1);
@@ -584,6 +643,59 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
         G.w_o = mat(g.o, W, g.heads * g.vdim);
         G.state_off = state;
         state += (long long)g.heads * g.dim * ((g.vdim + 7) / 8 * 8);   // value columns padded to eights, as for gated linear attention
+      } else if (ls.mixer == THA_MIX_WKV) {
+        const WkvSpec& g = ls.wkv;
+        if (g.heads < 1 || g.dim < 1) throw std::runtime_error("key-value memory: heads and dim must be positive");
+        if (g.dim > 512) throw std::runtime_error("key-value memory: more than 512 key channels per head are not served");
+        tha_wkv_t& G = L.wkv;
+        G.heads = g.heads; G.dim = g.dim; G.eps = spec.eps;
+        const TensorInfo& w1 = file.info(g.w1);
+        if (w1.shape.size() != 2) throw std::runtime_error("key-value memory: the decay projection must be a matrix");
+        G.rank = (int)w1.shape[0];
+        const long long hd = (long long)g.heads * g.dim;
+        G.o_r = in.add(g.r, hd);      // one grouped product, in this order
+        G.o_k = in.add(g.k, hd);
+        G.o_v = in.add(g.v, hd);
+        G.o_g = in.add(g.g, hd);
+        G.o_w1 = in.add(g.w1, G.rank);
+        std::vector<float> mu;
+        for (const std::string* n : {&g.mu_r, &g.mu_k, &g.mu_v, &g.mu_g, &g.mu_w}) {
+          const size_t before = mu.size();
+          file.read_f32(*n, &mu);
+          if (mu.size() != before + (size_t)W) throw std::runtime_error("tensor '" + *n + "': one value per channel of the width is expected");
+        }
+        G.mu = (const float*)m->upload(mu.data(), mu.size() * 4);
+        G.w_w2 = mat(g.w2, hd, G.rank);
+        G.w0 = vec(g.w0, (size_t)hd);
+        G.u = vec(g.u, (size_t)hd);
+        G.norm = vec(g.norm, (size_t)hd);
+        G.w_o = mat(g.o, W, (int)hd);
+        G.state_off = state;
+        state += tha_hyb_scan_state_floats(g.heads, g.dim, g.dim);
+        G.shift_state_off = state;
+        state += W;
+      } else if (ls.mixer == THA_MIX_RETENTION) {
+        const RetentionSpec& g = ls.retention;
+        if (g.heads < 1 || g.dim < 1 || g.vdim < 1) throw std::runtime_error("retention: heads, dim and vdim must be positive");
+        if (g.dim > 512) throw std::runtime_error("retention: more than 512 key channels per head are not served");
+        if ((int)g.decay.size() != g.heads) throw std::runtime_error("retention: one decay per head is expected");
+        tha_retention_t& G = L.retention;
+        G.heads = g.heads; G.dim = g.dim; G.vdim = g.vdim; G.eps = spec.eps;
+        G.rot = -1;
+        if (g.rotary && g.rot.dims > 0) {
+          if (g.rot.dims > g.dim || (g.rot.dims & 1)) throw std::runtime_error("retention: rotated dimensions must be even and at most dim");
+          G.rot = rotary(g.rot);
+          G.rot_layout = g.rot.halves ? THA_ROT_HALVES : THA_ROT_INTERLEAVED;
+        }
+        G.o_q = in.add(g.q, (long long)g.heads * g.dim);
+        G.o_k = in.add(g.k, (long long)g.heads * g.dim);
+        G.o_v = in.add(g.v, (long long)g.heads * g.vdim);
+        G.o_g = in.add(g.g, (long long)g.heads * g.vdim);
+        std::vector<float> dec(g.decay.begin(), g.decay.end());
+        G.decay = (const float*)m->upload(dec.data(), dec.size() * 4);
+        G.w_o = mat(g.o, W, g.heads * g.vdim);
+        G.state_off = state;
+        state += tha_hyb_scan_state_floats(g.heads, g.dim, g.vdim);
       } else if (ls.mixer == THA_MIX_LATENT) {
         const LatentSpec& a = ls.latent;
         const bool direct_q = !a.q.empty();
@@ -744,6 +856,19 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
       M.max_positions = spec.max_positions;
     }
     M.final_norm = norm(spec.final_norm);
+    if (spec.logit_scale != 1.0f) {
+      // the logits are linear in the final norm's output: its weight (and bias) carry their factor
+      std::vector<float> w, b;
+      file.read_f32(spec.final_norm, &w);
+      for (float& v : w) v = (M.final_norm.w_offset + v) * spec.logit_scale;
+      M.final_norm.w = (const float*)m->upload(w.data(), w.size() * 4);
+      M.final_norm.w_offset = 0.0f;
+      if (M.final_norm.b) {
+        file.read_f32(spec.final_norm + ".b", &b);
+        for (float& v : b) v *= spec.logit_scale;
+        M.final_norm.b = (const float*)m->upload(b.data(), b.size() * 4);
+      }
+    }
     M.head = mat(spec.head, spec.vocab, W);
     M.layers = m->layers_.data();
     M.n_rot = (int)m->rot_.size();

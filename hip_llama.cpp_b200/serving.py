@@ -457,3 +457,62 @@ def random_mozetar_tensors(cfg: dict, seed: int = 0) -> dict:
             a = 1.0 + 0.2 * rng.standard_normal(shape)
         out[name] = np.asarray(a, dtype=np.float32)
     return out
+
+
+def logulix_tensor_shapes(cfg: dict, decay_rank: int = 16) -> dict:
+    """name -> shape of every tensor a Logulix config asks for (decay_rank: rows of the key-value memory's first decay
+    projection, a property of the tensors and not of the config)."""
+    W, V = cfg["width"], cfg["vocab"]
+    s = {"embed": (V, W), "final.norm": (W,), "head": (V, W)}
+    if cfg.get("loop"):
+        s["loop.in"] = (W, 2 * W)
+    for i, L in enumerate(cfg["layers"]):
+        p, m, q = f"l{i}.", L["mixer"], f"l{i}.mix."
+        s[p + "norm1"] = (W,)
+        if L["type"] == "attention":
+            cq, ck = m["heads"] * m["dim"], m["kv_heads"] * m["dim"]
+            for n, c in (("q", cq), ("k", ck)):
+                s[q + n], s[q + n + ".b"], s[q + n + ".norm"] = (c, W), (c,), (c,)
+                if m.get("conv"):
+                    s[q + n + ".conv"] = (c, m["conv"])
+            s[q + "o"], s[q + "o.b"] = (W, cq), (W,)
+        elif L["type"] == "wkv":
+            c = m["heads"] * m["dim"]
+            for n in ("r", "k", "v", "g"):
+                s[q + n], s[q + "mu." + n] = (c, W), (W,)
+            s[q + "mu.w"], s[q + "w1"], s[q + "w2"], s[q + "w0"] = (W,), (decay_rank, W), (c, decay_rank), (c,)
+            s[q + "u"], s[q + "norm"], s[q + "o"] = (m["heads"], m["dim"]), (c,), (W, c)
+        elif L["type"] == "retention":
+            cq, cv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            s[q + "q"], s[q + "k"], s[q + "v"], s[q + "g"], s[q + "o"] = (cq, W), (cq, W), (cv, W), (cv, W), (W, cv)
+        else:
+            raise ValueError(L["type"])
+        f = L.get("mlp")
+        if f:
+            s[p + "norm2"], s[p + "mlp.up"], s[p + "mlp.down"] = (W,), (f["ff"], W), (W, f["ff"])
+    return s
+
+
+def random_logulix_tensors(cfg: dict, seed: int = 0, decay_rank: int = 16) -> dict:
+    """Random weights of a Logulix config: matrices N(0, 1/in), norm weights around one, small biases, convolution taps of
+    order one half, token-shift weights in (0, 1), decay offsets from slow to fast."""
+    rng = np.random.default_rng(seed)
+    out = {}
+    for name, shape in logulix_tensor_shapes(cfg, decay_rank).items():
+        last = name.rsplit(".", 1)[-1]
+        if last == "conv":
+            a = 0.5 * rng.standard_normal(shape)
+        elif last == "b":
+            a = 0.1 * rng.standard_normal(shape)
+        elif ".mu." in name:
+            a = rng.uniform(0.0, 1.0, shape)
+        elif last == "w0":
+            a = rng.uniform(-6.0, 0.0, shape)
+        elif last == "u":
+            a = 0.5 * rng.standard_normal(shape)
+        elif len(shape) == 2:
+            a = rng.standard_normal(shape, dtype=np.float32) * (1.0 if name == "embed" else 1.0 / np.sqrt(shape[1]))
+        else:
+            a = 1.0 + 0.2 * rng.standard_normal(shape)
+        out[name] = np.asarray(a, dtype=np.float32)
+    return out

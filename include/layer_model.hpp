@@ -27,9 +27,10 @@ struct RotarySpec {
   // l > original / low, between them (1 - s) f / factor + s f with s = (original / l - low) / (high - low); amplitude 1
   bool by_wavelength = false;
   double low = 1.0, high = 4.0;
+  bool linear = false;        // every frequency divided by `factor`
   bool operator==(const RotarySpec& o) const {
     return dims == o.dims && base == o.base && yarn == o.yarn && factor == o.factor && original == o.original && fast == o.fast &&
-           slow == o.slow && by_wavelength == o.by_wavelength && low == o.low && high == o.high;
+           slow == o.slow && by_wavelength == o.by_wavelength && low == o.low && high == o.high && linear == o.linear;
   }
 };
 struct AttnSpec {
@@ -53,11 +54,26 @@ struct AttnSpec {
   float q_temp_coef = 0.f;               // q_temp_every > 0: queries times 1 + coef * ln(floor((p + 1) / every) + 1)
   int q_temp_every = 0;
   int conv_taps = 0;                     // > 0: a short causal convolution behind the q, k and v projections ("<tensor>.conv")
+  std::string q_b, k_b, o_b;             // biases of the q, k and output projections; empty: none
+  std::string q_norm, k_norm;            // rms norms over the whole q row [heads * dim] and k row [kv_heads * dim]; empty: none
+  bool v_is_k = false;                   // no value tensor: the values are the keys as they leave the convolution (ahead of norm and rotation)
+  float softcap = 0.f;                   // > 0: scores s become softcap * tanh(s / softcap)
   int kv_from = -1;                      // >= 0: no key / value tensors; the layer reads the cache rows of that layer (index into `layers`)
 };
 struct HgrnSpec {
   int heads = 0, dim = 0, vdim = 0;
   std::string q, f, f_b, lower, v, norm, o;
+};
+struct WkvSpec {
+  int heads = 0, dim = 0;
+  std::string mu_r, mu_k, mu_v, mu_g, mu_w, r, k, v, g, w1, w2, w0, u, norm, o;   // the rank of w1 / w2 is read from the tensors
+};
+struct RetentionSpec {
+  int heads = 0, dim = 0, vdim = 0;
+  bool rotary = false;
+  RotarySpec rot;
+  std::vector<double> decay;             // [heads]
+  std::string q, k, v, g, o;
 };
 struct StreamsSpec {
   std::string in, out, mix;              // [n], [n], [n, n]
@@ -135,6 +151,9 @@ struct LayerSpec {
   bool pre_add_embed = false;            // before this run: x += the embedding output
   std::string pre_vec;                   // before this run: x += row pre_vec_row of this [rows, width] tensor; empty: none
   int pre_vec_row = 0;
+  std::string pre_join;                  // before this run: x <- (this [width, 2 * width] tensor) [x; embedding output]; empty: none
+  WkvSpec wkv;                           // THA_MIX_WKV
+  RetentionSpec retention;               // THA_MIX_RETENTION
   bool has_ff = false;
   MoeSpec moe;
   HgrnSpec hgrn;                         // THA_MIX_HGRN
@@ -151,6 +170,7 @@ struct LayerProgramSpec {
   float norm_w_offset = 1.0f;            // THA_NORM_RMS: what is added to the stored weight (0: the weight is stored as it is used)
   int n_streams = 0;                     // THA_BLOCK_STREAMS layers: copies of the residual
   float embed_scale = 1.0f;
+  float logit_scale = 1.0f;              // the logits' factor (taken into the final norm's weight)
   std::string side_table;                // [vocab, side_cols]: per-token side inputs, a column range per layer; empty: none
   int side_cols = 0;
   std::string pos_embed;                 // learned position vectors [max_positions, width]; empty: none

@@ -37,6 +37,8 @@ extern "C" {
 #define THA_MIX_ATTN 4     /* softmax attention alone (tha_attn_t with its window, sink, per-head scale and gate options) */
 #define THA_MIX_ATTN_GDELTA 5 /* softmax attention and a generalized delta rule side by side: mix_left * left + mix_right * right */
 #define THA_MIX_HGRN 6     /* gated linear recurrence whose forget gate also decides what is written (tha_hgrn_t) */
+#define THA_MIX_WKV 7      /* token-shifted key-value memory: decay per key channel, a bonus for the current token (tha_wkv_t) */
+#define THA_MIX_RETENTION 8 /* linear attention with one fixed decay per head (tha_retention_t) */
 
 #define THA_BLOCK_PARALLEL 0   /* x <- x + mixer(norm1 x) + ff(norm x): mixer and feed-forward read the same x */
 #define THA_BLOCK_SEQUENTIAL 1 /* x <- x + m mixer(norm1 x), then x <- x + m ff(norm2 x), then the per-token side input */
@@ -160,6 +162,15 @@ typedef struct {
   int conv_taps;
   const float* conv_w;
   long long conv_state_off;
+  const float* conv_b;     /* [channels] added to the projected channels ahead of the convolution (the tail keeps biased rows), NULL: none */
+  int v_is_k;              /* 1: no value projection; a value row is the key row as it leaves the convolution, ahead of norm and rotation
+                              (vdim == dim; o_v must equal o_k) */
+  /* row norms (NULL: none): the whole q row (all heads' channels, one mean) is divided by its root mean square and weighted, and the
+   * whole k row likewise, ahead of rotation; values are not normed */
+  const float* q_norm;     /* [heads * dim] */
+  const float* k_norm;     /* [kv_heads * dim] */
+  float softcap;           /* > 0: a scaled score s becomes softcap * tanh(s / softcap) ahead of the softmax */
+  const float* b_o;        /* [width] bias of the output projection (sequential blocks), NULL: none */
 } tha_attn_t;
 
 /* Generalized delta rule with a decay and a removal rate per key channel.  r, k, v, g: heads x dim columns each.
@@ -239,6 +250,38 @@ typedef struct {
   const void* w_o;      /* [width, heads * vdim] */
   long long state_off;
 } tha_hgrn_t;
+
+/* Token-shifted key-value memory.  With h' the previous token's normed input (zeros ahead of the first token), each of r, k, v, g and
+ * the decay input reads its own h + (h' - h) * mu; r, k, v: heads x dim columns each.
+ *   decay w = exp(-exp(W_w2 tanh(W_w1 mix_w) + w0)) per head and key channel
+ *   o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t,   S_t = diag(w_t) S_(t-1) + k_t v_t^T
+ * The read-out is divided by its root mean square per head, weighted (norm, [heads * dim]) and gated by silu(W_g mix_g).
+ * State: S per head laid out as for tha_gla_t; the last h (width floats). */
+typedef struct {
+  int heads, dim, rank;
+  float eps;
+  const float* mu;      /* [5, width]: r, k, v, g, decay */
+  int o_r, o_k, o_v, o_g, o_w1; /* columns of the grouped product (tha_hyb_linear_groups), in this order */
+  const void* w_w2;     /* [heads * dim, rank] */
+  const float* w0;      /* [heads * dim] */
+  const float* u;       /* [heads * dim] */
+  const float* norm;    /* [heads * dim] */
+  const void* w_o;      /* [width, heads * dim] */
+  long long state_off, shift_state_off;
+} tha_wkv_t;
+
+/* Retention.  q, k: heads x dim, v, gate: heads x vdim columns of the stacked projection; q and k rotated, k times dim^(-1/2).  Per head
+ * S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t with one fixed decay per head.  The read-out is divided by its root mean square
+ * per head (no weight) and gated by silu.  State per head as for tha_gla_t. */
+typedef struct {
+  int heads, dim, vdim;
+  int rot, rot_layout;  /* rotary table (-1: none), THA_ROT_* */
+  float eps;
+  int o_q, o_k, o_v, o_g;
+  const float* decay;   /* [heads] */
+  const void* w_o;      /* [width, heads * vdim] */
+  long long state_off;
+} tha_retention_t;
 
 /* Residual streams.  A model keeps n copies X[0..n-1] of its residual (all equal to the embedding output at the start).
  * A sublayer reads u = sum_s in[s] X[s], computes y = sublayer(norm(u)), and writes X'[t] = sum_s mix[s * n + t] X[s] + out[t] y
@@ -351,6 +394,10 @@ typedef struct {
   /* before this run's first norm: x += the embedding output (pre_add_embed), then x += pre_vec ([width], NULL: none) */
   int pre_add_embed;
   const float* pre_vec;
+  /* before this run's first norm (sequential blocks): x <- W_join [x; embedding output], [width, 2 * width], x first; NULL: none */
+  const void* w_join;
+  tha_wkv_t wkv;        /* THA_MIX_WKV */
+  tha_retention_t retention; /* THA_MIX_RETENTION */
   tha_hgrn_t hgrn;      /* THA_MIX_HGRN */
   /* THA_BLOCK_STREAMS: the two sublayers' stream weights; the feed-forward (dense or mixture, or none) reads norm2 through
    * w_in2.  in_conv_taps > 0: the mixer's normed input h is replaced by h + causal_conv(h) per channel (in_conv_w
@@ -405,6 +452,11 @@ int tha_hyb_norm_pair(void* stream, int dtype, void* out1, void* out2, const flo
 int tha_hyb_linear(void* stream, int dtype, float* C, long long ldc, const void* A, long long lda, int a_f32,
                    const int* a_rows, const void* W, long long w_group_stride, int M, int N, int K,
                    const int* group_off, int n_groups);
+/* n_groups products with an input of their own each, side by side: columns [sum of n before g, + group_n[g]) of C (row pitch ldc) =
+ * A_g . W_g^T, A_g = rows g * M .. g * M + M - 1 of A (dtype-typed, row pitch K), W_g the next group_n[g] rows of W [sum n, K].
+ * group_n is a host array; at most 8 groups. */
+int tha_hyb_linear_groups(void* stream, int dtype, float* C, long long ldc, const void* A, const void* W, int M, int K, int n_groups,
+                          const int* group_n_host);
 /* One product per head: C[m, h * c_hs + n] = sum_k A[m, h * a_hs + k] * W[h * w_hs + n * K + k], n < N, k < K, fp32 out.
  * a_f32: A is fp32 (else dtype-typed). */
 int tha_hyb_linear_heads(void* stream, int dtype, float* C, long long ldc, long long c_hs, const void* A, long long lda,
@@ -427,16 +479,17 @@ long long tha_hyb_gdelta_state_floats(int heads, int dim);
 /* out (dtype-typed [n_rows, side->dim]) = gelu_tanh(gate_raw) * table[token, side->col0 ..]: the input of the side projection */
 int tha_hyb_side_gate(void* stream, int dtype, void* out, const float* gate_raw, long long ldg, const tha_side_t* side,
                       const void* side_table, int side_cols, const int* token, int n_rows);
-/* the end of a sequential block, one pass over x: x += m * ff (ff NULL: none); x += m * y / sqrt(mean(y^2) + eps) * y_norm
+/* the end of a sequential block, one pass over x: x += m * (ff + ff_b) (ff NULL: none; ff_b [width] NULL: no bias); x += m * y / sqrt(mean(y^2) + eps) * y_norm
  * (y NULL: none); tap (nullable) receives x; then x += embed_out (nullable), x += vec (nullable), and with next_norm not
- * NULL out (dtype-typed) = that norm of x -- what comes ahead of the next layer run */
-int tha_hyb_block_finish(void* stream, int dtype, float* x, const float* ff, const float* y, float m, const float* y_norm, float eps,
-                         float* tap, const float* embed_out, const float* vec, const tha_norm_t* next_norm, void* out, int n_rows,
-                         int width);
-/* x += c_left * left + c_right * right (right NULL: none) (+ embed_out when given) (+ vec when given); then, with n not NULL,
- * out (dtype-typed) = the norm n of x (THA_NORM_COPY: x itself).  left NULL: only the optional addends. */
-int tha_hyb_add_norm(void* stream, int dtype, float* x, const float* left, float c_left, const float* right, float c_right,
-                     const float* embed_out, const float* vec, const tha_norm_t* n, float eps, void* out, int n_rows, int width);
+ * NULL out (dtype-typed, row pitch ldo; 0: width) = that norm of x -- what comes ahead of the next layer run */
+int tha_hyb_block_finish(void* stream, int dtype, float* x, const float* ff, const float* ff_b, const float* y, float m, const float* y_norm, float eps,
+                         float* tap, const float* embed_out, const float* vec, const tha_norm_t* next_norm, void* out, long long ldo,
+                         int n_rows, int width);
+/* x += c_left * (left + left_b) + c_right * right (left_b, right NULL: none) (+ embed_out when given) (+ vec when given); then, with n not NULL,
+ * out (dtype-typed, row pitch ldo; 0: width) = the norm n of x (THA_NORM_COPY: x itself).  left NULL: only the optional addends. */
+int tha_hyb_add_norm(void* stream, int dtype, float* x, const float* left, const float* left_b, float c_left, const float* right,
+                     float c_right, const float* embed_out, const float* vec, const tha_norm_t* n, float eps, void* out, long long ldo,
+                     int n_rows, int width);
 /* softmax attention of every row over its visible cache rows; out dtype-typed [n_rows, heads * vdim].
  * split_scratch (nullable, fp32): room for the partial results when a step of few rows at long contexts is cut along
  * the keys (splits * n_rows * heads * (vdim + 2) floats are used, as many splits as fit, at most 16) */
@@ -469,7 +522,7 @@ int tha_hyb_latent_prepare(void* stream, int dtype, const tha_latent_t* a, const
 int tha_hyb_latent_split_q(void* stream, int dtype, const tha_latent_t* a, int n_rows, const float* qfull, long long ldq,
                            const float* cos_t, const float* sin_t, int rot_dims, void* q_plain, float* q_abs);
 /* out (dtype-typed [n_rows, heads * E]) = o_raw * gate_act(gate) (gate NULL: no gate), with do_norm: o_raw divided by its rms per head and
- * weighted by norm ([E], or [heads * E] with norm_per_head) first */
+ * weighted by norm ([E], or [heads * E] with norm_per_head; NULL: no weight) first */
 int tha_hyb_head_gate(void* stream, int dtype, void* out, const float* o_raw, int n_rows, int heads, int E, int do_norm,
                       float eps, const float* norm, int norm_per_head, const float* gate, long long ldg, int gate_act);
 /* gated linear attention over the rows of every sequence in order: z_raw [n_rows, heads * dim] (W_a2 a1, before the bias)
@@ -490,12 +543,28 @@ int tha_hyb_ff_act(void* stream, int dtype, int act, void* y, const float* gu, l
 
 /* causal convolution over `channels` adjacent columns of proj starting at col0, continuing from the slot's tail (the last
  * taps - 1 inputs of every channel): out[r, c] = act(sum_j w[c, j] in(r - taps + 1 + j, c)) (+ in(r, c) with add_input);
+ * bias ([channels], NULL: none) is added to the step's rows before they meet the taps; the tail holds rows with it.
  * act 0: none, 1: silu.  out fp32 [n_rows, channels] (out_f32) or dtype-typed.  The tails are NOT advanced (tha_hyb_conv_tail). */
 int tha_hyb_conv(void* stream, int dtype, const tha_rows_t* rows, const tha_state_store_t* st, long long conv_state_off, const float* proj,
-                 long long ldp, int col0, int channels, int taps, const float* w, int act, int add_input, int out_f32, void* out);
+                 long long ldp, int col0, int channels, int taps, const float* w, const float* bias, int act, int add_input, int out_f32,
+                 void* out);
 /* the tails of a convolution advanced by the step's rows */
 int tha_hyb_conv_tail(void* stream, const tha_rows_t* rows, const tha_state_store_t* st, long long conv_state_off, const float* proj,
-                      long long ldp, int col0, int channels, int taps);
+                      long long ldp, int col0, int channels, int taps, const float* bias);
+/* token shift: out [n_mix][n_rows, width] (dtype-typed), out[i, r] = h[r] + (h_prev - h[r]) * mu[i], h_prev the sequence's row before r
+ * (in the step, else the slot's width floats at shift_state_off); then the slots keep every sequence's last row */
+int tha_hyb_token_shift(void* stream, int dtype, const tha_rows_t* rows, const tha_state_store_t* st, long long shift_state_off, const float* h,
+                        int width, const float* mu, int n_mix, void* out);
+/* the token-shifted key-value memory over the rows of every sequence in order, proj = the grouped product of the five mixes: decay
+ * [n_rows, heads * dim] receives the decays; the read-out goes to o_raw (fp32) and, normed, weighted and gated, to out (dtype-typed) */
+int tha_hyb_wkv_scan(void* stream, int dtype, const tha_wkv_t* g, const tha_rows_t* rows, const tha_state_store_t* st, const float* proj,
+                     long long ldp, float* decay, float* o_raw, void* out);
+/* retention over the rows of every sequence in order: the q and k columns of proj are rotated (k scaled) in place; the read-out goes to
+ * o_raw (fp32 [n_rows, heads * vdim]) and, normed and gated, to out (dtype-typed) */
+int tha_hyb_retention_scan(void* stream, int dtype, const tha_retention_t* g, const tha_rows_t* rows, const tha_state_store_t* st, float* proj,
+                           long long ldp, const float* cos_t, const float* sin_t, int rot_dims, float* o_raw, void* out);
+/* floats of one sequence's state of a scanned memory (tha_gla_t, tha_hgrn_t, tha_wkv_t, tha_retention_t) */
+long long tha_hyb_scan_state_floats(int heads, int dim, int vdim);
 /* Residual streams, one pass over the rows.  X [n_rows, n, width] fp32.  init (nullable): every stream is first set to
  * init [n_rows, width].  write (nullable): X'[t] = sum_s write->mix[s, t] X[s] + write->out[t] * y, where
  * y = dense (nullable) + bias (nullable) + sum_j weight[r, j] * down[inv[r, j]] (top picks of a mixture; top 0: none).

@@ -9,6 +9,7 @@ import numpy as np
 import pytest
 
 import bozovik_oracle as B
+import logulix_oracle as L
 import mozetar_oracle as M
 import numizen_oracle as N
 import timerax_oracle as O
@@ -43,7 +44,7 @@ def test_registry_names_what_it_knows(tmp_path):
     with pytest.raises(serving.ServingError) as e:
         serving.ServingEngine(str(tmp_path), "float32", 64, 1)
     assert "Nope" in str(e.value) and "Timerax" in str(e.value) and "llama2" in str(e.value) and "Numizen" in str(e.value)
-    assert "Bozovik" in str(e.value) and "Mozetar" in str(e.value)
+    assert "Bozovik" in str(e.value) and "Mozetar" in str(e.value) and "Logulix" in str(e.value)
 
 
 @built
@@ -352,3 +353,74 @@ def test_plain_mozetar_convolution_recurrence_and_router():
     # PolyNorm: each power is normed by itself, so scaling the input leaves everything but the constant's share unchanged
     z = np.array([[1.0, -2.0, 3.0]])
     assert np.allclose(M.polynorm(z, [0.5, 0.3, 0.2, 0.1], 0.0), M.polynorm(7.0 * z, [0.5, 0.3, 0.2, 0.1], 0.0))
+
+
+# ---- Logulix ----------------------------------------------------------------------------------------------------------
+def _logulix_cfg(layers, **extra):
+    c = {"architecture": "Logulix", "width": 16, "vocab": 20, "norm": {"eps": 1e-5}, "embedding": {"scale": 2.0}, "logit_scale": 0.5, "layers": layers}
+    c.update(extra)
+    return c
+
+
+@built
+def test_logulix_configs_are_refused_by_name(tmp_path):
+    serving = load_pkg("serving")
+    att = {"type": "attention", "mlp": None, "mixer": {"heads": 2, "kv_heads": 1, "dim": 4, "vdim": 4, "scale": 0.5, "softcap": 9.0, "conv": 2,
+                                                       "mask": {"size": 3}}}
+    ret = {"type": "retention", "mixer": {"heads": 2, "dim": 4, "vdim": 6}, "mlp": None}
+    for cfg, word in [(_logulix_cfg([{"type": "helix", "mixer": {}, "mlp": None}]), "helix"),
+                      (_logulix_cfg([dict(att, mlp={"kind": "sparse"})]), "sparse"),
+                      (_logulix_cfg([ret]), "decay"),
+                      (_logulix_cfg([dict(att, mixer=dict(att["mixer"], mask={"size": 0}))]), "window"),
+                      (_logulix_cfg([dict(att, mixer=dict(att["mixer"], conv=0))]), "conv"),
+                      (_logulix_cfg([dict(att, mixer=dict(att["mixer"], softcap=0.0))]), "softcap"),
+                      (_logulix_cfg([att], loop={"start": 0, "stop": 2, "times": 2}), "loop"),
+                      ({k: v for k, v in _logulix_cfg([att]).items() if k != "logit_scale"}, "logit_scale")]:
+        (tmp_path / "config.json").write_text(json.dumps(cfg))
+        with pytest.raises(serving.ServingError) as e:
+            serving.ServingEngine(str(tmp_path), "float32", 64, 1)
+        assert word in str(e.value), (word, str(e.value))
+
+
+def test_logulix_tensor_shapes_cover_a_config():
+    serving = load_pkg("serving")
+    layers = [{"type": "attention", "mixer": {"heads": 4, "kv_heads": 2, "dim": 6, "vdim": 6, "scale": 0.4, "softcap": 5.0, "conv": 3, "mask": {"size": 7}},
+               "mlp": {"kind": "dense", "ff": 12}},
+              {"type": "wkv", "mixer": {"heads": 2, "dim": 5}, "mlp": None},
+              {"type": "retention", "mixer": {"heads": 2, "dim": 3, "vdim": 7, "decay": [0.5, 0.9]}, "mlp": {"kind": "dense", "ff": 9}}]
+    cfg = _logulix_cfg(layers, loop={"start": 1, "stop": 3, "times": 2})
+    t = serving.random_logulix_tensors(cfg, 0, decay_rank=3)
+    assert t["l0.mix.q"].shape == (24, 16) and t["l0.mix.k"].shape == (12, 16) and t["l0.mix.k.conv"].shape == (12, 3) and "l0.mix.v" not in t
+    assert t["l0.mix.q.norm"].shape == (24,) and t["l0.mix.o.b"].shape == (16,) and t["loop.in"].shape == (16, 32)
+    assert t["l1.mix.w1"].shape == (3, 16) and t["l1.mix.w2"].shape == (10, 3) and t["l1.mix.u"].shape == (2, 5) and "l1.norm2" not in t
+    assert t["l2.mix.v"].shape == (14, 16) and t["l2.mix.q"].shape == (6, 16) and t["l2.mlp.up"].shape == (9, 16)
+    assert {k: v.shape for k, v in t.items()} == L.tensor_shapes(cfg, 3)
+
+
+def test_plain_logulix_statements_agree():
+    assert L.self_check()
+
+
+def test_plain_logulix_runs_bonus_and_values():
+    runs = L.layer_runs({"layers": [0, 0, 0, 0], "loop": {"start": 1, "stop": 3, "times": 2}})
+    assert runs == [(0, False), (1, True), (2, False), (1, True), (2, False), (3, False)]
+    # one head of one channel, mixes off: o_1 = u k v r, o_2 = (k1 v1 + u k2 v2) r2; the stored state carries no bonus
+    W = {n: np.eye(1) for n in "rkvg"}
+    W.update({"mu." + c: np.zeros(1) for c in "rkvgw"})
+    W.update({"w1": np.zeros((1, 1)), "w2": np.zeros((1, 1)), "w0": np.full(1, -40.0), "u": np.full((1, 1), 3.0), "norm": np.ones(1), "o": np.eye(1)})
+    st = {}
+    L.wkv_mixer(np.array([[2.0], [5.0]]), {"heads": 1, "dim": 1}, {"p." + k: v for k, v in W.items()}, "p.", 1e-6, st)
+    assert np.allclose(st["S"], 4.0 + 25.0) and np.allclose(st["h"], 5.0)
+    # rotations pair (i, i + dims / 2) or neighbours; entries from `dims` on pass; a linear stretch slows the angle
+    x = np.arange(6, dtype=np.float64).reshape(1, 1, 6)
+    r = {"dims": 4, "base": 1.0, "scaling": {"factor": 2.0}}
+    a, b = L.rotate(x, [1], r, True)[0, 0], L.rotate(x, [1], r, False)[0, 0]
+    c, s = np.cos(0.5), np.sin(0.5)
+    assert np.allclose(a, [0 * c - 2 * s, 1 * c - 3 * s, 2 * c + 0 * s, 3 * c + 1 * s, 4, 5])
+    assert np.allclose(b, [0 * c - 1 * s, 1 * c + 0 * s, 2 * c - 3 * s, 3 * c + 2 * s, 4, 5])
+    # values are the convolved keys: with one visible key (window 1) the read-out is that row, whatever the norms and scores
+    m = {"heads": 2, "kv_heads": 1, "dim": 2, "conv": 2, "scale": 1.0, "softcap": 1.0, "mask": {"size": 1}}
+    W = {"q": np.ones((4, 2)), "k": np.eye(2), "q.b": np.zeros(4), "k.b": np.array([1.0, 0.0]), "q.conv": np.ones((4, 2)), "k.conv": np.array([[10.0, 1.0]] * 2),
+         "q.norm": np.ones(4), "k.norm": np.ones(2), "o": np.eye(4)[:2], "o.b": np.array([0.5, 0.0])}
+    y = L.attention_mixer(np.array([[1.0, 2.0], [3.0, 4.0]]), m, {"p." + k: v for k, v in W.items()}, "p.", 1e-6, {}, 0)
+    assert np.allclose(y, [[2.0 + 0.5, 2.0], [20.0 + 4.0 + 0.5, 20.0 + 4.0]])
