@@ -3,7 +3,9 @@ Numizen beside Timerax -- the closest design the framework has: attention + a re
 and llama2 at equal size (bench.py --design numizen); or of Bozovik beside Numizen with dense feed-forwards -- the closest
 design the framework has: latent attention + a recurrent mixer + a looped segment -- and llama2 at equal size (bench.py
 --design bozovik); or of Mozetar beside Numizen -- the closest design the framework has: softmax attention + a gated linear
-recurrence + a mixture of experts behind a softmax router with groups -- and llama2 at equal size (bench.py --design mozetar).
+recurrence + a mixture of experts behind a softmax router with groups -- and llama2 at equal size (bench.py --design mozetar);
+or of Logulix beside Bozovik (sequential blocks, windowed attention, a recurrent mixer, ungated dense feed-forwards, a looped segment),
+Numizen with dense feed-forwards (the scan its memories share) and llama2 at equal size (bench.py --design logulix).
 
 Random weights at sizes that resemble a real model's layers; a few layers only, so that building the folder stays
 short.  For every size: prompt ingestion (one prompt in one step) and batched decoding (one token per live request per
@@ -117,6 +119,27 @@ def mozetar_config(s: dict, n: dict) -> dict:
     layers = [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": dense if i == 0 else moe} for i in range(s["layers"])]
     return {"architecture": "Mozetar", "layers": layers, "norm": {"eps": 1e-6}, "canon": {"taps": 3}, "streams": 3, "vocab": s["vocab"],
             "width": s["width"]}
+
+
+# Logulix at the same widths and vocabulary: retention, windowed attention with keys as values, the token-shifted key-value memory, and
+# retention again; layers 1 and 2 are a looped segment that runs once (so its joining map runs); retention heads as Numizen's linear
+# attention, key-value memory heads of 64 over the whole width; the ungated feed-forward of the Bozovik arm.
+LOGULIX = {
+    "w1024": dict(window=1024, rheads=4, rdim=128, rvdim=256, wheads=16, wdim=64),
+    "w2048": dict(window=2048, rheads=8, rdim=128, rvdim=256, wheads=32, wdim=64),
+}
+
+
+def logulix_config(s: dict, n: dict) -> dict:
+    att = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "conv": 4, "scale": s["dim"] ** -0.5, "softcap": 50.0,
+           "mask": {"size": n["window"]}, "rot": {"base": 500000.0, "dims": s["dim"], "scaling": {"factor": 2.0}}}
+    ret = {"heads": n["rheads"], "dim": n["rdim"], "vdim": n["rvdim"], "rot": {"base": 500000.0, "dims": n["rdim"]},
+           "decay": [1.0 - 2.0 ** -(5 + i) for i in range(n["rheads"])]}
+    mlp = {"kind": "dense", "ff": (s["top"] * s["ff"] + s["sff"]) * 3 // 2}
+    kinds = [("retention", ret), ("attention", att), ("wkv", {"heads": n["wheads"], "dim": n["wdim"]}), ("retention", ret)]
+    layers = [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": mlp} for i in range(s["layers"])]
+    return {"architecture": "Logulix", "layers": layers, "norm": {"eps": 1e-6}, "vocab": s["vocab"], "width": s["width"],
+            "embedding": {"scale": 1.0}, "logit_scale": 0.5, "loop": {"start": 1, "stop": min(3, s["layers"]), "times": 1}}
 
 
 def _time_timerax(serving, folder, prompt_len, batch, ctx, steps, warmup, kernels):
@@ -250,6 +273,27 @@ def run(load_pkg, sizes, prompt_len=4096, batch=64, ctx=512, steps=16, warmup=3,
     for name in sizes:
         s = SIZES[name]
         r = {}
+        if design == "logulix":
+            def arm(cfg, tensors, shapes):
+                tmp = tempfile.mkdtemp(prefix="design_bench_")
+                try:
+                    serving.save_model_folder(tmp, cfg, tensors)
+                    out = _time_folder(serving, tmp, prompt_len, batch, ctx, steps, warmup, kernels)
+                    out["weights_bytes"] = timerax_weight_bytes(cfg, shapes)
+                    return out
+                finally:
+                    shutil.rmtree(tmp, ignore_errors=True)
+            c = logulix_config(s, LOGULIX[name])
+            r["logulix"] = arm(c, serving.random_logulix_tensors(c, 0, decay_rank=64), serving.logulix_tensor_shapes(c, 64))
+            if not kernels or llama:
+                c = bozovik_config(s, BOZOVIK[name])
+                r["bozovik"] = arm(c, serving.random_bozovik_tensors(c, 0, decay_rank=64), serving.bozovik_tensor_shapes(c, 64))
+                c = numizen_config(s, NUMIZEN[name], max_positions=max(prompt_len, ctx + steps + warmup) + 64, dense_everywhere=True)
+                r["numizen_dense"] = arm(c, serving.random_numizen_tensors(c, 0), serving.numizen_tensor_shapes(c))
+            if llama and not kernels:
+                r["llama2_bf16_equal_size"] = _time_llama(engine_mod, checkpoint_mod, s, prompt_len, batch, ctx, steps, warmup)
+            results[name] = r
+            continue
         if design == "mozetar":
             mcfg = mozetar_config(s, MOZETAR[name])
             tmp = tempfile.mkdtemp(prefix="design_bench_")

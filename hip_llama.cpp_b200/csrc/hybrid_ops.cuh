@@ -32,9 +32,10 @@ __device__ __forceinline__ float hyb_rotated(const float* src, int d, int rot_di
 
 // The scanned memories (hybrid_gla.cu): forms of the recurrence and the launch they share.  dec [n_rows, heads * dim]: decays per key
 // channel (not SCAN_HEAD_DECAY); aux: [heads] decays (SCAN_HEAD_DECAY) or [heads * dim] bonus (SCAN_BONUS).
+// scratch (nullable): tha_hyb_scan_scratch_floats, lets long portions run as segments side by side.
 enum { SCAN_CHANNEL_DECAY = 0, SCAN_HEAD_DECAY = 1, SCAN_BONUS = 2 };
 int hyb_scan_launch(cudaStream_t s, int form, const tha_gla_t* g, const tha_rows_t* rows, const tha_state_store_t* st, const float* proj, long long ldp,
-                    const float* dec, const float* aux, float* o_raw, float qscale);
+                    const float* dec, const float* aux, float* o_raw, float qscale, float* scratch, size_t scratch_floats);
 
 // first float of the cache row of (slot, position t) in cache layer `layer` of a pool
 __device__ __forceinline__ size_t hyb_kv_row(const tha_kv_t& kv, int slot, int t, int layer) {

@@ -39,7 +39,7 @@ __global__ void hyb_rotate_qk_kernel(float* __restrict__ proj, long long ldp, in
 using namespace tha;
 
 extern "C" int tha_hyb_retention_scan(void* stream, int dtype, const tha_retention_t* g, const tha_rows_t* rows, const tha_state_store_t* st,
-                                      float* proj, long long ldp, const float* cos_t, const float* sin_t, int rot_dims, float* o_raw, void* out) {
+                                      float* proj, long long ldp, const float* cos_t, const float* sin_t, int rot_dims, float* o_raw, void* out, float* seg_scratch, size_t seg_scratch_floats) {
   if (rows->n_seqs < 1 || rows->n_rows < 1) return THA_STATUS_SUCCESS;
   if (g->heads < 1 || g->dim < 1 || g->vdim < 1 || rot_dims > g->dim || (rot_dims & 1)) return THA_STATUS_INVALID_ARG;
   if (g->dim > 512) return THA_STATUS_NOT_SUPPORTED;
@@ -48,7 +48,7 @@ extern "C" int tha_hyb_retention_scan(void* stream, int dtype, const tha_retenti
                      g->rot_layout, cos_t, sin_t, 1.0f / sqrtf((float)g->dim)));
   tha_gla_t a = {};
   a.heads = g->heads; a.dim = g->dim; a.vdim = g->vdim; a.o_q = g->o_q; a.o_k = g->o_k; a.o_v = g->o_v; a.state_off = g->state_off;
-  const int status = hyb_scan_launch(s, SCAN_HEAD_DECAY, &a, rows, st, proj, ldp, nullptr, g->decay, o_raw, 1.0f);
+  const int status = hyb_scan_launch(s, SCAN_HEAD_DECAY, &a, rows, st, proj, ldp, nullptr, g->decay, o_raw, 1.0f, seg_scratch, seg_scratch_floats);
   if (status != THA_STATUS_SUCCESS) return status;
   return tha_hyb_head_gate(stream, dtype, out, o_raw, rows->n_rows, g->heads, g->vdim, 1, g->eps, nullptr, 0, proj + g->o_g, ldp, THA_GATE_SILU);
 }

@@ -101,6 +101,7 @@ struct StepBuffers {
   float *proj2, *qfull, *x0, *sgate;
   float *xs, *hf, *att;   // the residual streams [rows, n, width]; a normed input before its convolution; fp32 attention maps
   void* sg;
+  float* scan; size_t scan_floats;   // segments of the scanned memories in long portions
   void *join, *mix;        // the joining map's input [rows, 2 width]; the token-shifted inputs [5][rows, width]
   void *h, *h2, *cq, *qplain, *abuf, *mbuf, *y, *sy, *hn, *hg;
   int *expert_id, *group_off, *sorted_row, *inv;
@@ -125,13 +126,17 @@ static size_t hyb_attn_conv_channels(const tha_attn_t& a) {
   return c;
 }
 
-static size_t carve(const tha_hyb_model_t* m, int R, int n_want, char* base, StepBuffers* b) {
+static size_t carve(const tha_hyb_model_t* m, const tha_rows_t* rows, int n_want, char* base, StepBuffers* b) {
+  const int R = rows->n_rows;
   Carver c{base};
   const size_t W = m->width, es = m->dtype == THA_DT_BF16 ? 2 : 4;
   size_t n_in = 0, qd = 0, av = 0, mv = 0, cc = 0, dd = 0, dg = 0, gu = 0, ff = 0, sff = 0, top = 0, ne = 0;
   size_t n_in2 = 0, qr = 0, qf = 0, qp = 0;
   bool norm2 = false, keep_embed = false, join = false, shift = false;
-  size_t sd = 0, n_str = 0, hfw = 0, attf = 0;
+  size_t sd = 0, n_str = 0, hfw = 0, attf = 0, scan = 0;
+  auto scan_scratch = [&](int heads, int dim, int vdim) {
+    scan = max(scan, tha_hyb_scan_scratch_floats(heads, dim, vdim, rows->n_rows, rows->n_seqs, rows->max_seq_rows));
+  };
   for (int i = 0; i < m->n_layers; i++) {
     const tha_hyb_layer_t& L = m->layers[i];
     n_in = max(n_in, (size_t)L.n_in);
@@ -149,14 +154,19 @@ static size_t carve(const tha_hyb_model_t* m, int R, int n_want, char* base, Ste
     if (L.mixer == THA_MIX_HGRN) {
       dd = max(dd, (size_t)L.hgrn.heads * L.hgrn.dim);
       mv = max(mv, (size_t)L.hgrn.heads * L.hgrn.vdim);
+      scan_scratch(L.hgrn.heads, L.hgrn.dim, L.hgrn.vdim);
     }
     if (L.mixer == THA_MIX_WKV) {
       shift = true;
       hfw = W;
       dd = max(dd, (size_t)L.wkv.heads * L.wkv.dim);
       mv = max(mv, (size_t)L.wkv.heads * L.wkv.dim);
+      scan_scratch(L.wkv.heads, L.wkv.dim, L.wkv.dim);
     }
-    if (L.mixer == THA_MIX_RETENTION) mv = max(mv, (size_t)L.retention.heads * L.retention.vdim);
+    if (L.mixer == THA_MIX_RETENTION) {
+      mv = max(mv, (size_t)L.retention.heads * L.retention.vdim);
+      scan_scratch(L.retention.heads, L.retention.dim, L.retention.vdim);
+    }
     if (L.mixer == THA_MIX_ATTN_GDELTA) {
       dd = max(dd, (size_t)L.gdelta.heads * L.gdelta.dim);
       mv = max(mv, (size_t)L.gdelta.heads * L.gdelta.dim);
@@ -173,6 +183,7 @@ static size_t carve(const tha_hyb_model_t* m, int R, int n_want, char* base, Ste
     } else if (L.mixer == THA_MIX_GLA) {
       dd = max(dd, (size_t)L.gla.heads * L.gla.dim);
       mv = max(mv, (size_t)L.gla.heads * L.gla.vdim);
+      scan_scratch(L.gla.heads, L.gla.dim, L.gla.vdim);
     } else if (L.mixer == THA_MIX_LATENT) {
       const tha_latent_t& a = L.latent;
       qr = max(qr, (size_t)a.q_rank);
@@ -215,6 +226,8 @@ static size_t carve(const tha_hyb_model_t* m, int R, int n_want, char* base, Ste
   // key splits of the attention in small steps: 16 x rows x heads x (vdim + 2) floats at most (2 * heads <= 2 * heads * dim)
   b->split_floats = R <= 1024 ? (size_t)16 * R * (av + 2 * qd) : 0;
   b->split = c.take<float>(b->split_floats);
+  b->scan_floats = scan;
+  b->scan = scan ? c.take<float>(scan) : nullptr;
   b->left = c.take<float>(R * W);
   b->right = c.take<float>(R * W);
   b->conv = c.take<float>(R * cc);
@@ -305,7 +318,7 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
   HybScratch& sc = g_scratch[dev & 63];
   std::lock_guard<std::mutex> lock(sc.mu);
   StepBuffers b;
-  const size_t need = carve(m, R, n_want, nullptr, &b);
+  const size_t need = carve(m, rows, n_want, nullptr, &b);
   if (need > sc.cap) {   // grow: nothing of an earlier step may still be using the old slab
     THA_CUDA_OK(cudaDeviceSynchronize());
     if (sc.base) THA_CUDA_OK(cudaFree(sc.base));
@@ -314,7 +327,7 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
     THA_CUDA_OK(cudaMalloc((void**)&sc.base, want));
     sc.cap = want;
   }
-  carve(m, R, n_want, sc.base, &b);
+  carve(m, rows, n_want, sc.base, &b);
 
   const float embed_scale = m->embed_scale != 0.f ? m->embed_scale : 1.0f;
   if (dt == THA_DT_BF16)
@@ -430,20 +443,20 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
     } else if (L.mixer == THA_MIX_GLA) {
       const tha_gla_t& g = L.gla;
       HYB_OK(tha_hyb_linear(stream, dt, b.dt_raw, g.heads * g.dim, b.proj + g.o_a1, ldp, 1, nullptr, g.w_a2, 0, R, g.heads * g.dim, g.rank, nullptr, 0));
-      HYB_OK(tha_hyb_gla_scan(stream, dt, &g, rows, st, b.proj, ldp, b.dt_raw, b.oraw, b.mbuf));
+      HYB_OK(tha_hyb_gla_scan(stream, dt, &g, rows, st, b.proj, ldp, b.dt_raw, b.oraw, b.mbuf, b.scan, b.scan_floats));
       HYB_OK(tha_hyb_linear(stream, dt, b.left, W, b.mbuf, g.heads * g.vdim, 0, nullptr, g.w_o, 0, R, W, g.heads * g.vdim, nullptr, 0));
     } else if (L.mixer == THA_MIX_HGRN) {
       const tha_hgrn_t& g = L.hgrn;
-      HYB_OK(tha_hyb_hgrn_scan(stream, dt, &g, rows, st, b.proj, ldp, b.dt_raw, b.oraw, b.mbuf));
+      HYB_OK(tha_hyb_hgrn_scan(stream, dt, &g, rows, st, b.proj, ldp, b.dt_raw, b.oraw, b.mbuf, b.scan, b.scan_floats));
       HYB_OK(tha_hyb_linear(stream, dt, b.left, W, b.mbuf, g.heads * g.vdim, 0, nullptr, g.w_o, 0, R, W, g.heads * g.vdim, nullptr, 0));
     } else if (L.mixer == THA_MIX_WKV) {
       const tha_wkv_t& g = L.wkv;
-      HYB_OK(tha_hyb_wkv_scan(stream, dt, &g, rows, st, b.proj, ldp, b.dt_raw, b.oraw, b.mbuf));
+      HYB_OK(tha_hyb_wkv_scan(stream, dt, &g, rows, st, b.proj, ldp, b.dt_raw, b.oraw, b.mbuf, b.scan, b.scan_floats));
       HYB_OK(tha_hyb_linear(stream, dt, b.left, W, b.mbuf, g.heads * g.dim, 0, nullptr, g.w_o, 0, R, W, g.heads * g.dim, nullptr, 0));
     } else if (L.mixer == THA_MIX_RETENTION) {
       const tha_retention_t& g = L.retention;
       HYB_OK(tha_hyb_retention_scan(stream, dt, &g, rows, st, b.proj, ldp, g.rot >= 0 ? b.cos_t[g.rot] : nullptr, g.rot >= 0 ? b.sin_t[g.rot] : nullptr,
-                                    g.rot >= 0 ? m->rot[g.rot].dims : 0, b.oraw, b.mbuf));
+                                    g.rot >= 0 ? m->rot[g.rot].dims : 0, b.oraw, b.mbuf, b.scan, b.scan_floats));
       HYB_OK(tha_hyb_linear(stream, dt, b.left, W, b.mbuf, g.heads * g.vdim, 0, nullptr, g.w_o, 0, R, W, g.heads * g.vdim, nullptr, 0));
     } else if (L.mixer == THA_MIX_LATENT) {
       const tha_latent_t& a = L.latent;

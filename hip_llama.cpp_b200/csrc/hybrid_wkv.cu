@@ -118,7 +118,7 @@ extern "C" int tha_hyb_token_shift(void* stream, int dtype, const tha_rows_t* ro
 }
 
 extern "C" int tha_hyb_wkv_scan(void* stream, int dtype, const tha_wkv_t* g, const tha_rows_t* rows, const tha_state_store_t* st,
-                                const float* proj, long long ldp, float* decay, float* o_raw, void* out) {
+                                const float* proj, long long ldp, float* decay, float* o_raw, void* out, float* seg_scratch, size_t seg_scratch_floats) {
   if (rows->n_seqs < 1 || rows->n_rows < 1) return THA_STATUS_SUCCESS;
   if (g->heads < 1 || g->dim < 1 || g->rank < 1) return THA_STATUS_INVALID_ARG;
   if (g->dim > 512) return THA_STATUS_NOT_SUPPORTED;
@@ -131,7 +131,7 @@ extern "C" int tha_hyb_wkv_scan(void* stream, int dtype, const tha_wkv_t* g, con
     THA_CUDA_OK(launch(hyb_wkv_decay_kernel<float>, grid, dim3(256), 0, s, false, decay, proj + g->o_w1, ldp, g->rank, (const float*)g->w_w2, g->w0, R, HD));
   tha_gla_t a = {};
   a.heads = g->heads; a.dim = g->dim; a.vdim = g->dim; a.o_q = g->o_r; a.o_k = g->o_k; a.o_v = g->o_v; a.state_off = g->state_off;
-  const int status = hyb_scan_launch(s, SCAN_BONUS, &a, rows, st, proj, ldp, decay, g->u, o_raw, 1.0f);
+  const int status = hyb_scan_launch(s, SCAN_BONUS, &a, rows, st, proj, ldp, decay, g->u, o_raw, 1.0f, seg_scratch, seg_scratch_floats);
   if (status != THA_STATUS_SUCCESS) return status;
   return tha_hyb_head_gate(stream, dtype, out, o_raw, R, g->heads, g->dim, 1, g->eps, g->norm, 1, proj + g->o_g, ldp, THA_GATE_SILU);
 }

@@ -528,7 +528,7 @@ int tha_hyb_head_gate(void* stream, int dtype, void* out, const float* o_raw, in
 /* gated linear attention over the rows of every sequence in order: z_raw [n_rows, heads * dim] (W_a2 a1, before the bias)
  * is replaced by the decays; the read-out goes to o_raw (fp32 [n_rows, heads * vdim]) and, normed and gated, to out */
 int tha_hyb_gla_scan(void* stream, int dtype, const tha_gla_t* g, const tha_rows_t* rows, const tha_state_store_t* st,
-                     const float* proj, long long ldp, float* z_raw, float* o_raw, void* out);
+                     const float* proj, long long ldp, float* z_raw, float* o_raw, void* out, float* seg_scratch, size_t seg_scratch_floats);
 /* router: expert ids and weights [n_rows, top]; rows sorted by expert: group_off (2 * (experts + 1) ints: the offsets,
  * then scratch), sorted_row [n_rows * top] and the position of (row, j) in that order, inv [n_rows * top] */
 int tha_hyb_moe_route(void* stream, const tha_moe_t* e, const float* proj, long long ldp, int n_rows, int* expert_id,
@@ -558,13 +558,16 @@ int tha_hyb_token_shift(void* stream, int dtype, const tha_rows_t* rows, const t
 /* the token-shifted key-value memory over the rows of every sequence in order, proj = the grouped product of the five mixes: decay
  * [n_rows, heads * dim] receives the decays; the read-out goes to o_raw (fp32) and, normed, weighted and gated, to out (dtype-typed) */
 int tha_hyb_wkv_scan(void* stream, int dtype, const tha_wkv_t* g, const tha_rows_t* rows, const tha_state_store_t* st, const float* proj,
-                     long long ldp, float* decay, float* o_raw, void* out);
+                     long long ldp, float* decay, float* o_raw, void* out, float* seg_scratch, size_t seg_scratch_floats);
 /* retention over the rows of every sequence in order: the q and k columns of proj are rotated (k scaled) in place; the read-out goes to
  * o_raw (fp32 [n_rows, heads * vdim]) and, normed and gated, to out (dtype-typed) */
 int tha_hyb_retention_scan(void* stream, int dtype, const tha_retention_t* g, const tha_rows_t* rows, const tha_state_store_t* st, float* proj,
-                           long long ldp, const float* cos_t, const float* sin_t, int rot_dims, float* o_raw, void* out);
+                           long long ldp, const float* cos_t, const float* sin_t, int rot_dims, float* o_raw, void* out, float* seg_scratch,
+                           size_t seg_scratch_floats);
 /* floats of one sequence's state of a scanned memory (tha_gla_t, tha_hgrn_t, tha_wkv_t, tha_retention_t) */
 long long tha_hyb_scan_state_floats(int heads, int dim, int vdim);
+/* floats of the scratch (seg_scratch of the scans above, NULL: none) with which a step's long portions run as segments side by side */
+size_t tha_hyb_scan_scratch_floats(int heads, int dim, int vdim, int n_rows, int n_seqs, int max_seq_rows);
 /* Residual streams, one pass over the rows.  X [n_rows, n, width] fp32.  init (nullable): every stream is first set to
  * init [n_rows, width].  write (nullable): X'[t] = sum_s write->mix[s, t] X[s] + write->out[t] * y, where
  * y = dense (nullable) + bias (nullable) + sum_j weight[r, j] * down[inv[r, j]] (top picks of a mixture; top 0: none).
@@ -583,7 +586,7 @@ int tha_hyb_diff_combine(void* stream, int dtype, const tha_attn_t* a, const flo
 /* the bounded-forget-gate recurrence over the rows of every sequence in order: the q columns of proj are replaced by their silu,
  * the f columns by 1 - f, decay [n_rows, heads * dim] receives f; read-out to o_raw (fp32), normed to out (dtype-typed) */
 int tha_hyb_hgrn_scan(void* stream, int dtype, const tha_hgrn_t* g, const tha_rows_t* rows, const tha_state_store_t* st, float* proj,
-                      long long ldp, float* decay, float* o_raw, void* out);
+                      long long ldp, float* decay, float* o_raw, void* out, float* seg_scratch, size_t seg_scratch_floats);
 
 #ifdef __cplusplus
 }
