@@ -76,7 +76,16 @@ __device__ __forceinline__ ScanPlace scan_place(const tha_rows_t& rows, int len,
   return p;
 }
 
-template <int RPL, int AHEAD, int GLA_COLS, int FORM, bool LOCAL>
+// VEC consecutive floats (one 32-, 64- or 128-bit load; the caller checks the alignment)
+template <int VEC> __device__ __forceinline__ void scan_ld(const float* p, float* o) {
+  if (VEC == 4) { const float4 t = *reinterpret_cast<const float4*>(p); o[0] = t.x; o[1] = t.y; o[2] = t.z; o[3] = t.w; }
+  else if (VEC == 2) { const float2 t = *reinterpret_cast<const float2*>(p); o[0] = t.x; o[1] = t.y; }
+  else o[0] = *p;
+}
+
+// VEC: consecutive key channels per lane (lane l owns l * VEC .. of every run of 32 * VEC; VEC > 1 needs dim, offsets and row pitches
+// that are multiples of it, and of four value columns), so that a lane's inputs are few wide loads
+template <int RPL, int AHEAD, int GLA_COLS, int FORM, bool LOCAL, int VEC>
 __global__ void __launch_bounds__(32 * GLA_WARPS) hyb_gla_scan_kernel(tha_gla_t g, tha_rows_t rows, tha_state_store_t st,
                                                                       const float* __restrict__ proj, long long ldp,
                                                                       const float* __restrict__ decay, const float* __restrict__ aux,
@@ -94,21 +103,44 @@ __global__ void __launch_bounds__(32 * GLA_WARPS) hyb_gla_scan_kernel(tha_gla_t 
   const float* start = at.n_seg == 1 || (LOCAL && at.seg == 0) ? slot
                        : segs.states + (size_t)(at.entry + (at.seg == 0 ? at.n_seg - 1 : at.seg - 1)) * entry + mine;
   const bool from_zero = LOCAL && at.seg > 0;
+  const bool pairs = ((reinterpret_cast<size_t>(slot) | reinterpret_cast<size_t>(segs.states)) & 7) == 0;
+  auto ch = [&](int i) { return (i / VEC) * (32 * VEC) + lane * VEC + i % VEC; };   // this lane's i-th key channel
+  // a column pair of a channel is one 64-bit word where the regions start on even floats (the loader's do); one branch outside, so
+  // that all of a lane's loads are in flight together
   float S[RPL][GLA_COLS];
+  if (pairs) {
+    float2 t[RPL][GLA_COLS / 2];
 #pragma unroll
-  for (int i = 0; i < RPL; i++) {
-    const int d = lane + 32 * i;
+    for (int i = 0; i < RPL; i++)
 #pragma unroll
-    for (int c = 0; c < GLA_COLS; c++) S[i][c] = (d < D && e0 + c < E && !from_zero) ? start[(size_t)(c >> 1) * 2 * D + 2 * d + (c & 1)] : 0.f;
-  }
-  auto leave = [&](float* dst) {
+      for (int c = 0; c < GLA_COLS; c += 2) {
+        const bool live = ch(i) < D && e0 + c < E && !from_zero;
+        t[i][c / 2] = live ? *reinterpret_cast<const float2*>(start + (size_t)c * D + 2 * ch(i)) : make_float2(0.f, 0.f);
+      }
 #pragma unroll
-    for (int i = 0; i < RPL; i++) {
-      const int d = lane + 32 * i;
-      if (d >= D) continue;
+    for (int i = 0; i < RPL; i++)
+#pragma unroll
+      for (int c = 0; c < GLA_COLS; c += 2) { S[i][c] = t[i][c / 2].x; S[i][c + 1] = e0 + c + 1 < E ? t[i][c / 2].y : 0.f; }
+  } else {
+#pragma unroll
+    for (int i = 0; i < RPL; i++)
 #pragma unroll
       for (int c = 0; c < GLA_COLS; c++)
-        if (e0 + c < E) dst[(size_t)(c >> 1) * 2 * D + 2 * d + (c & 1)] = S[i][c];
+        S[i][c] = (ch(i) < D && e0 + c < E && !from_zero) ? start[(size_t)(c >> 1) * 2 * D + 2 * ch(i) + (c & 1)] : 0.f;
+  }
+  auto leave = [&](float* dst) {
+    if (pairs) {
+#pragma unroll
+      for (int i = 0; i < RPL; i++)
+#pragma unroll
+        for (int c = 0; c < GLA_COLS; c += 2)   // an odd last column's partner is padding
+          if (ch(i) < D && e0 + c < E) *reinterpret_cast<float2*>(dst + (size_t)c * D + 2 * ch(i)) = make_float2(S[i][c], S[i][c + 1]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < RPL; i++)
+#pragma unroll
+        for (int c = 0; c < GLA_COLS; c++)
+          if (ch(i) < D && e0 + c < E) dst[(size_t)(c >> 1) * 2 * D + 2 * ch(i) + (c & 1)] = S[i][c];
     }
   };
   if (LOCAL && at.seg == 0) leave(segs.states + (size_t)(at.entry + at.n_seg - 1) * entry + mine);
@@ -117,7 +149,7 @@ __global__ void __launch_bounds__(32 * GLA_WARPS) hyb_gla_scan_kernel(tha_gla_t 
   if (FORM == SCAN_HEAD_DECAY) fixed_decay = aux[h];
   if (BONUS) {
 #pragma unroll
-    for (int i = 0; i < RPL; i++) bonus[i] = lane + 32 * i < D ? aux[h * D + lane + 32 * i] : 0.f;
+    for (int i = 0; i < RPL; i++) bonus[i] = ch(i) < D ? aux[h * D + ch(i)] : 0.f;
   }
   if (LOCAL) {
 #pragma unroll
@@ -130,14 +162,33 @@ __global__ void __launch_bounds__(32 * GLA_WARPS) hyb_gla_scan_kernel(tha_gla_t 
   auto fetch = [&](int r, In& in) {
     const float* x = proj + (size_t)r * ldp;
 #pragma unroll
-    for (int i = 0; i < RPL; i++) {
-      const int d = lane + 32 * i;
-      if (!LOCAL) in.q[i] = d < D ? x[g.o_q + h * D + d] : 0.f;
-      in.k[i] = d < D ? x[g.o_k + h * D + d] : 0.f;
-      if (FORM != SCAN_HEAD_DECAY) in.a[i] = d < D ? decay[(size_t)r * g.heads * D + h * D + d] : 0.f;
-    }
+    for (int i = 0; i < RPL; i += VEC) {
+      const int d = ch(i);
+      if (d < D) {
+        if (!LOCAL) scan_ld<VEC>(x + g.o_q + h * D + d, in.q + i);
+        scan_ld<VEC>(x + g.o_k + h * D + d, in.k + i);
+        if (FORM != SCAN_HEAD_DECAY) scan_ld<VEC>(decay + (size_t)r * g.heads * D + h * D + d, in.a + i);
+      } else {
 #pragma unroll
-    for (int c = 0; c < GLA_COLS; c++) in.v[c] = e0 + c < E ? x[g.o_v + h * E + e0 + c] : 0.f;
+        for (int v = i; v < i + VEC; v++) {
+          if (!LOCAL) in.q[v] = 0.f;
+          in.k[v] = 0.f;
+          if (FORM != SCAN_HEAD_DECAY) in.a[v] = 0.f;
+        }
+      }
+    }
+    if (VEC > 1) {
+#pragma unroll
+      for (int c = 0; c < GLA_COLS; c += 4) {
+        if (e0 + c < E) scan_ld<4>(x + g.o_v + h * E + e0 + c, in.v + c);
+        else
+#pragma unroll
+          for (int v = 0; v < 4; v++) in.v[c + v] = 0.f;
+      }
+    } else {
+#pragma unroll
+      for (int c = 0; c < GLA_COLS; c++) in.v[c] = e0 + c < E ? x[g.o_v + h * E + e0 + c] : 0.f;
+    }
   };
 #pragma unroll
   for (int u = 0; u < AHEAD; u++)
@@ -212,7 +263,7 @@ __global__ void __launch_bounds__(32 * GLA_WARPS) hyb_gla_scan_kernel(tha_gla_t 
     if (e0 == 0) {
 #pragma unroll
       for (int i = 0; i < RPL; i++)
-        if (lane + 32 * i < D) segs.prods[(size_t)(at.entry + at.seg) * g.heads * D + h * D + lane + 32 * i] = prod[i];
+        if (ch(i) < D) segs.prods[(size_t)(at.entry + at.seg) * g.heads * D + h * D + ch(i)] = prod[i];
     }
   } else if (at.seg == at.n_seg - 1) {
     leave(slot);
@@ -284,18 +335,26 @@ static int gla_scan_launch(cudaStream_t s, const tha_gla_t* g, const tha_rows_t*
     }
   }
   const bool seg = segs.len > 0;
-  const int cols = seg && g->dim <= 128 ? 4 : 2;
+  const int vec = g->dim <= 32 ? 1 : g->dim <= 64 ? 2 : 4;
+  const bool wide = seg && g->dim > 32 && g->dim <= 128 && g->dim % vec == 0 && g->o_q % vec == 0 && g->o_k % vec == 0 && ldp % 4 == 0 && g->o_v % 4 == 0 &&
+                    g->vdim % 4 == 0 && aligned16(proj) && (!dec || aligned16(dec));
+  const bool decode = !seg && rows->max_seq_rows <= 2 && g->dim <= 128;
+  const int cols = wide ? 8 : (seg || decode) && g->dim <= 128 ? 4 : 2;
   const dim3 grid(seg ? rows->n_rows / len + rows->n_seqs : rows->n_seqs, g->heads, ceil_div(g->vdim, cols * GLA_WARPS)), block(32 * GLA_WARPS);
-#define GLA_LAUNCH(R, A, C, F, L) THA_CUDA_OK(launch(hyb_gla_scan_kernel<R, A, C, F, L>, grid, block, 0, s, false, *g, *rows, *st, proj, ldp, dec, aux, o_raw, qscale, segs))
-#define GLA_BOTH(R, A, C) do { if (seg) { GLA_LAUNCH(R, A, C, LFORM, true); \
+#define GLA_LAUNCH(R, A, C, F, L, V) THA_CUDA_OK(launch(hyb_gla_scan_kernel<R, A, C, F, L, V>, grid, block, 0, s, false, *g, *rows, *st, proj, ldp, dec, aux, o_raw, qscale, segs))
+#define GLA_BOTH(R, A, C, V) do { if (seg) { GLA_LAUNCH(R, A, C, LFORM, true, V); \
     THA_CUDA_OK(launch(hyb_scan_combine_kernel, dim3(ceil_div(g->dim * ((g->vdim + GLA_STATE_PAD - 1) / GLA_STATE_PAD * GLA_STATE_PAD), 256), g->heads, rows->n_seqs), \
                        dim3(256), 0, s, false, *g, *rows, segs)); } \
-    GLA_LAUNCH(R, A, C, FORM, false); } while (0)
-  if (g->dim <= 32) { if (cols == 4) GLA_BOTH(1, 4, 4); else GLA_BOTH(1, 4, 2); }
-  else if (g->dim <= 64) { if (cols == 4) GLA_BOTH(2, 4, 4); else GLA_BOTH(2, 4, 2); }
-  else if (g->dim <= 128) { if (cols == 4) GLA_BOTH(4, 4, 4); else GLA_BOTH(4, 4, 2); }
-  else if (g->dim <= 256) GLA_BOTH(8, 2, 2);
-  else GLA_BOTH(16, 1, 2);
+    GLA_LAUNCH(R, A, C, FORM, false, V); } while (0)
+  // many warps per scheduler (segments): wide loads, eight columns a warp, two tokens ahead; few: two columns, four tokens ahead
+  if (wide) { if (g->dim <= 64) GLA_BOTH(2, 2, 8, 2); else GLA_BOTH(4, 2, 8, 4); }
+  // decoding: nearly all of it is reading and writing states, so many warps with few registers each
+  else if (decode) { if (g->dim <= 32) GLA_LAUNCH(1, 1, 4, FORM, false, 1); else if (g->dim <= 64) GLA_LAUNCH(2, 1, 4, FORM, false, 1); else GLA_LAUNCH(4, 1, 4, FORM, false, 1); }
+  else if (g->dim <= 32) { if (cols == 4) GLA_BOTH(1, 4, 4, 1); else GLA_BOTH(1, 4, 2, 1); }
+  else if (g->dim <= 64) { if (cols == 4) GLA_BOTH(2, 4, 4, 1); else GLA_BOTH(2, 4, 2, 1); }
+  else if (g->dim <= 128) { if (cols == 4) GLA_BOTH(4, 4, 4, 1); else GLA_BOTH(4, 4, 2, 1); }
+  else if (g->dim <= 256) GLA_BOTH(8, 2, 2, 1);
+  else GLA_BOTH(16, 1, 2, 1);
 #undef GLA_BOTH
 #undef GLA_LAUNCH
   return THA_STATUS_SUCCESS;

@@ -446,6 +446,7 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
         if (!ls.pre_vec.empty()) L.pre_vec = pre_vector(ls.pre_vec, ls.pre_vec_row);
         if (L.in_conv_taps > 1) { L.in_conv_state_off = state; state += (long long)W * (L.in_conv_taps - 1); }
         if (L.mixer == THA_MIX_HGRN) {
+          state = (state + 3) / 4 * 4;
           L.hgrn.state_off = state;
           state += (long long)L.hgrn.heads * L.hgrn.dim * ((L.hgrn.vdim + 7) / 8 * 8);
         }
@@ -460,12 +461,14 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
           state += C * (A.conv_taps - 1);
         }
         if (L.mixer == THA_MIX_WKV) {
+          state = (state + 3) / 4 * 4;
           L.wkv.state_off = state;
           state += tha_hyb_scan_state_floats(L.wkv.heads, L.wkv.dim, L.wkv.dim);
           L.wkv.shift_state_off = state;
           state += W;
         }
         if (L.mixer == THA_MIX_RETENTION) {
+          state = (state + 3) / 4 * 4;
           L.retention.state_off = state;
           state += tha_hyb_scan_state_floats(L.retention.heads, L.retention.dim, L.retention.vdim);
         }
@@ -485,6 +488,7 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
           L.delta.conv_state_off = state;
           state += (2ll * L.delta.kv_heads * L.delta.dim + (long long)L.delta.heads * L.delta.vdim) * (L.delta.taps - 1);
         } else if (L.mixer == THA_MIX_GLA) {
+          state = (state + 3) / 4 * 4;
           L.gla.state_off = state;
           state += (long long)L.gla.heads * L.gla.dim * ((L.gla.vdim + 7) / 8 * 8);   // value columns padded to eights
         } else if (L.mixer == THA_MIX_LATENT) {
@@ -552,6 +556,7 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
           G.a_b = vec(g.a_b, (size_t)hd);
           G.norm = vec(g.norm, (size_t)hd);
           G.w_o = mat(g.o, W, (int)hd);
+          state = (state + 3) / 4 * 4;
           G.state_off = state;
           state += tha_hyb_gdelta_state_floats(g.heads, g.dim);
           L.mix_left = ls.mix_left; L.mix_right = ls.mix_right;
@@ -626,6 +631,7 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
         G.b_a2 = vec(g.a2_b, (size_t)g.heads * g.dim);
         G.norm = vec(g.norm, g.vdim);
         G.w_o = mat(g.o, W, g.heads * g.vdim);
+        state = (state + 3) / 4 * 4;
         G.state_off = state;
         state += (long long)g.heads * g.dim * ((g.vdim + 7) / 8 * 8);   // value columns padded to eights
       } else if (ls.mixer == THA_MIX_HGRN) {
@@ -641,6 +647,7 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
         G.lower = vec(g.lower, (size_t)g.heads * g.dim);
         G.norm = vec(g.norm, g.vdim);
         G.w_o = mat(g.o, W, g.heads * g.vdim);
+        state = (state + 3) / 4 * 4;
         G.state_off = state;
         state += (long long)g.heads * g.dim * ((g.vdim + 7) / 8 * 8);   // value columns padded to eights, as for gated linear attention
       } else if (ls.mixer == THA_MIX_WKV) {
@@ -670,6 +677,7 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
         G.u = vec(g.u, (size_t)hd);
         G.norm = vec(g.norm, (size_t)hd);
         G.w_o = mat(g.o, W, (int)hd);
+        state = (state + 3) / 4 * 4;
         G.state_off = state;
         state += tha_hyb_scan_state_floats(g.heads, g.dim, g.dim);
         G.shift_state_off = state;
@@ -694,6 +702,7 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
         std::vector<float> dec(g.decay.begin(), g.decay.end());
         G.decay = (const float*)m->upload(dec.data(), dec.size() * 4);
         G.w_o = mat(g.o, W, g.heads * g.vdim);
+        state = (state + 3) / 4 * 4;
         G.state_off = state;
         state += tha_hyb_scan_state_floats(g.heads, g.dim, g.vdim);
       } else if (ls.mixer == THA_MIX_LATENT) {
@@ -833,7 +842,7 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
         L.w_in2 = m->upload(in2.data(), in2.bytes());
       }
     }
-    m->state_floats_ = state > 0 ? state : 1;
+    m->state_floats_ = state > 0 ? (state + 3) / 4 * 4 : 4;   // whole 16-byte words: the scans read their states in wide words
     if (m->rot_.size() > 64) throw std::runtime_error("more than 64 distinct rotary tables");
     tha_hyb_model_t& M = m->model_;
     M.dtype = dtype;

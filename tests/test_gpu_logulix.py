@@ -252,6 +252,24 @@ def test_retention_long_prompts_and_portions(tmp_path, dim, vdim):
     check_all_positions(b, n=400, cuts=[300, 1], dtype="bfloat16", tol=BF16_TOL)
 
 
+@pytest.mark.parametrize("dim", [24, 64, 128])
+def test_long_and_short_portions_in_one_batch(tmp_path, dim):
+    """long portions run as segments side by side, short ones and single tokens in the same step do not: every sequence continues from
+    its own state, before and after"""
+    b = Built(tmp_path, model([wkv(heads=2, dim=dim), retention(heads=2, dim=dim, vdim=dim + 8, rot=None, decay=(0.9, 0.999))], width=48, vocab=90), 8)
+    lens = {"a": (5, 390, 1, 200), "b": (1, 64, 1, 1), "c": (40, 260, 3, 1), "d": (2, 1, 300, 2)}
+    toks = {k: tokens_for(b, sum(v), 70 + i) for i, (k, v) in enumerate(lens.items())}
+    e, got, at = b.engine(max_tokens=2048), {k: [] for k in lens}, dict.fromkeys(lens, 0)
+    for i in range(4):
+        out, o = e.step([(k, toks[k][at[k]:at[k] + v[i]], list(range(v[i]))) for k, v in lens.items()]), 0
+        for k, v in lens.items():
+            got[k].append(out[o:o + v[i]])
+            o += v[i]
+            at[k] += v[i]
+    for k in lens:
+        assert rel_err(np.concatenate(got[k]), b.ref(toks[k])[0]) < F32_TOL, k
+
+
 @pytest.mark.parametrize("loop", [(0, 1, 2), (0, 3, 2), (1, 3, 4), (2, 3, 1), (1, 2, 3)])
 def test_looped_segment(tmp_path, loop):
     """at the start, at the end, over everything, one layer, one pass; the map that joins x with the embedding output runs once a pass"""

@@ -250,6 +250,13 @@ def test_portions_bfloat16(general):
     assert rel_err(got, z) < BF16_TOL
 
 
+def test_long_prompts_whose_memories_run_as_segments(general):
+    toks = tokens_for(general, 420, 17)
+    z, _ = general.ref(toks)
+    for cuts in ([420], [17, 300, 1, 2], [200, 210]):
+        assert rel_err(feed(general.engine(), "a", toks, cuts), z) < F32_TOL
+
+
 def test_long_decoding(general):
     toks = tokens_for(general, 330, 9)
     z, _ = general.ref(toks)
