@@ -4,10 +4,10 @@
 // whose embedding rows and logits are multiplied by constants.
 // Layer types:
 //   "attention"  sliding-window softmax attention without a value projection: q and k carry biases and a short convolution, the values
-//                are the keys as they leave it; rms norms over the whole q and k rows, rotary pairs (2i, 2i + 1) with linearly
+//                are the convolved keys, not normed or rotated; rms norms over the whole q and k rows, rotary pairs (2i, 2i + 1) with linearly
 //                stretched frequencies, capped scores, an output bias;
 //   "wkv"        a token-shifted key-value memory: decay per key channel, a bonus for the current token, head norm, silu gate;
-//   "retention"  linear attention with one fixed decay per head, rotary pairs (i, i + dims / 2), head norm without a weight, silu gate.
+//   "retention"  a linear-attention memory whose only decay is a constant per head, rotary pairs (i, i + dims / 2), head norm without a weight, silu gate.
 // Feed-forward: none, or dense without a gate and with squared relu.
 // "loop" runs a segment of the layer list several times with the same weights, every pass with a cache and state of its own; every
 // pass starts by joining x and the embedding output through one map.  Every size and constant comes from the config; constants the

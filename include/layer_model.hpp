@@ -56,7 +56,7 @@ struct AttnSpec {
   int conv_taps = 0;                     // > 0: a short causal convolution behind the q, k and v projections ("<tensor>.conv")
   std::string q_b, k_b, o_b;             // biases of the q, k and output projections; empty: none
   std::string q_norm, k_norm;            // rms norms over the whole q row [heads * dim] and k row [kv_heads * dim]; empty: none
-  bool v_is_k = false;                   // no value tensor: the values are the keys as they leave the convolution (ahead of norm and rotation)
+  bool v_is_k = false;                   // no value tensor: values are the convolved keys, not normed or rotated
   float softcap = 0.f;                   // > 0: scores s become softcap * tanh(s / softcap)
   int kv_from = -1;                      // >= 0: no key / value tensors; the layer reads the cache rows of that layer (index into `layers`)
 };

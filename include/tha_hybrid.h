@@ -38,7 +38,7 @@ extern "C" {
 #define THA_MIX_ATTN_GDELTA 5 /* softmax attention and a generalized delta rule side by side: mix_left * left + mix_right * right */
 #define THA_MIX_HGRN 6     /* gated linear recurrence whose forget gate also decides what is written (tha_hgrn_t) */
 #define THA_MIX_WKV 7      /* token-shifted key-value memory: decay per key channel, a bonus for the current token (tha_wkv_t) */
-#define THA_MIX_RETENTION 8 /* linear attention with one fixed decay per head (tha_retention_t) */
+#define THA_MIX_RETENTION 8 /* linear-attention memory whose only decay is a constant per head (tha_retention_t) */
 
 #define THA_BLOCK_PARALLEL 0   /* x <- x + mixer(norm1 x) + ff(norm x): mixer and feed-forward read the same x */
 #define THA_BLOCK_SEQUENTIAL 1 /* x <- x + m mixer(norm1 x), then x <- x + m ff(norm2 x), then the per-token side input */
@@ -163,7 +163,7 @@ typedef struct {
   const float* conv_w;
   long long conv_state_off;
   const float* conv_b;     /* [channels] added to the projected channels ahead of the convolution (the tail keeps biased rows), NULL: none */
-  int v_is_k;              /* 1: no value projection; a value row is the key row as it leaves the convolution, ahead of norm and rotation
+  int v_is_k;              /* 1: no value projection; each value row is the convolved key row, not normed or rotated
                               (vdim == dim; o_v must equal o_k) */
   /* row norms (NULL: none): the whole q row (all heads' channels, one mean) is divided by its root mean square and weighted, and the
    * whole k row likewise, ahead of rotation; values are not normed */

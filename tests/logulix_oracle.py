@@ -58,7 +58,7 @@ def rotate(x, pos, rot, halves):
 
 # ---- mixers -------------------------------------------------------------------------------------------------------------
 def attention_mixer(h, m, W, p, eps, store, pos0):
-    """Softmax attention under a sliding window; the values are the keys as they leave the convolution."""
+    """Softmax attention under a sliding window; values are the convolved, not yet normed or rotated keys."""
     T = h.shape[0]
     H, G, D = m["heads"], m["kv_heads"], m["dim"]
     pos = pos0 + np.arange(T)
