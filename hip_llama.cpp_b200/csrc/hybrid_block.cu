@@ -7,6 +7,8 @@
 //   hyb_side_gate_kernel    gelu_tanh of the side gate's product times the token's entries of the side table
 //   hyb_block_finish_kernel x += m * ff, x += m * y / rms(y) * w for the side projection y, the layer's tap, then the addends
 //                           and the first norm of the NEXT layer run: one pass over x at the end of a block.
+//   hyb_post_norm_kernel    the end of a post-norm sublayer (THA_BLOCK_POST): the sublayer's result is put together (a product, a mixture's
+//                           picks, both), divided by its root mean square, weighted and added to x, which the next product gets a copy of.
 // The two side products themselves are the framework's matrix products (tha_hyb_linear).
 // The residual stream, the norms, the gate's activation and the side norm are fp32 in both number formats; sums run in a
 // fixed order per row, so a row's result does not depend on the rest of the step.
@@ -122,6 +124,51 @@ __global__ void hyb_block_finish_kernel(float* __restrict__ x, const float* __re
   }
 }
 
+// V channels per thread and step (4: width a multiple of four); the row of y waits in shared memory for its root mean square
+template <typename T, int V>
+__global__ void hyb_post_norm_kernel(float* __restrict__ x, const float* __restrict__ dense, const float* __restrict__ dense_gate, long long ldg, int top,
+                                     const float* __restrict__ weight, const int* __restrict__ inv, const float* __restrict__ down, float m, tha_norm_t n,
+                                     float eps, float* __restrict__ tap, T* __restrict__ out, int width) {
+  extern __shared__ __align__(16) float yrow[];
+  __shared__ float red[33];
+  const size_t r = blockIdx.x;
+  const float sg = dense_gate ? hyb_sigmoid(dense_gate[r * ldg]) : 1.0f;
+  float ss = 0.f;
+  for (int c = V * threadIdx.x; c < width; c += V * blockDim.x) {
+    float y[V];
+#pragma unroll
+    for (int v = 0; v < V; v++) y[v] = 0.f;
+    if (dense) {
+      hyb_load_vec(dense + r * width + c, y);
+#pragma unroll
+      for (int v = 0; v < V; v++) y[v] *= sg;
+    }
+#pragma unroll 4
+    for (int j = 0; j < top; j++) {
+      float d[V];
+      const float w = weight[r * top + j];
+      hyb_load_vec(down + (size_t)inv[r * top + j] * width + c, d);
+#pragma unroll
+      for (int v = 0; v < V; v++) y[v] = fmaf(w, d[v], y[v]);
+    }
+#pragma unroll
+    for (int v = 0; v < V; v++) { yrow[c + v] = y[v]; ss = fmaf(y[v], y[v], ss); }
+  }
+  ss = block_sum(ss, red);
+  const float f = m / sqrtf(ss / (float)width + eps);
+  // every thread reads back only what it wrote itself
+  for (int c = V * threadIdx.x; c < width; c += V * blockDim.x) {
+    float xv[V], wv[V];
+    hyb_load_vec(x + r * width + c, xv);
+    hyb_load_vec(n.w + c, wv);
+#pragma unroll
+    for (int v = 0; v < V; v++) xv[v] = fmaf(yrow[c + v] * f, n.w_offset + wv[v], xv[v]);
+    hyb_store_vec(x + r * width + c, xv);
+    if (tap) hyb_store_vec(tap + r * width + c, xv);
+    if (out) hyb_store_vec(out + r * width + c, xv);
+  }
+}
+
 }  // namespace tha
 
 using namespace tha;
@@ -176,5 +223,26 @@ extern "C" int tha_hyb_block_finish(void* stream, int dtype, float* x, const flo
   else
     THA_CUDA_OK(launch(hyb_block_finish_kernel<float>, dim3(n_rows), dim3(nt), 0, (cudaStream_t)stream, false, x, ff, ff_b, y, m, y_norm, eps, tap, embed_out,
                        vec, next_norm ? *next_norm : none, next_norm ? 1 : 0, (float*)out, ldo > 0 ? ldo : (long long)width, width));
+  return THA_STATUS_SUCCESS;
+}
+
+extern "C" int tha_hyb_post_norm(void* stream, int dtype, float* x, const float* dense, const float* dense_gate, long long ldg, int top,
+                                 const float* weight, const int* inv, const float* down, float m, const tha_norm_t* norm, float eps, float* tap,
+                                 void* out, int n_rows, int width) {
+  if (n_rows < 1) return THA_STATUS_SUCCESS;
+  if (!x || !norm || norm->kind != THA_NORM_RMS || !norm->w || (top > 0 && (!weight || !inv || !down))) return THA_STATUS_INVALID_ARG;
+  const size_t smem = sizeof(float) * (size_t)width;
+  if (smem > 220 * 1024) return THA_STATUS_NOT_SUPPORTED;
+  const bool vec = width % 4 == 0 && aligned16(x) && aligned16(dense) && aligned16(down) && aligned16(norm->w) && aligned16(tap) && aligned16(out);
+  const dim3 grid(n_rows), block(block_threads(width));
+#define POST_GO(T, V)                                                                                                                     \
+  do {                                                                                                                                    \
+    if (smem > 47 * 1024) THA_CUDA_OK(cudaFuncSetAttribute(hyb_post_norm_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+    THA_CUDA_OK(launch(hyb_post_norm_kernel<T, V>, grid, block, smem, (cudaStream_t)stream, false, x, dense, dense_gate, ldg, top, weight, inv, down, m, \
+                       *norm, eps, tap, (T*)out, width));                                                                                 \
+  } while (0)
+  if (dtype == THA_DT_BF16) { if (vec) POST_GO(bf16, 4); else POST_GO(bf16, 1); }
+  else { if (vec) POST_GO(float, 4); else POST_GO(float, 1); }
+#undef POST_GO
   return THA_STATUS_SUCCESS;
 }

@@ -287,7 +287,7 @@ __global__ void hyb_attn_prepare_kernel(tha_attn_t a, tha_rows_t rows, tha_kv_t 
   const float q_mult = a.q_temp_every > 0 ? 1.0f + a.q_temp_coef * logf((float)((t + 1) / a.q_temp_every + 1)) : 1.0f;
   // row norms: one mean over all heads' channels, taken by the whole block before the heads are dealt to its warps
   float row_q = 1.0f, row_k = 1.0f;
-  if (a.q_norm || a.k_norm) {
+  if (!a.head_norm && (a.q_norm || a.k_norm)) {
     __shared__ float red[33];
     if (a.q_norm) {
       float ss = 0.f;
@@ -301,8 +301,15 @@ __global__ void hyb_attn_prepare_kernel(tha_attn_t a, tha_rows_t rows, tha_kv_t 
     }
   }
   for (int h = warp; h < a.heads + n_k + n_v; h += nwarps) {
-    if (h >= a.heads + n_k) {   // a value head: plain copy
+    if (h >= a.heads + n_k) {   // a value head: plain copy, or blended with an earlier layer's values of the token
       const int g = h - a.heads - n_k;
+      if (a.v_mix) {
+        const float* first = kv.v_pool + hyb_kv_row(kv, slot, t, a.v_mix_layer) + (size_t)g * a.vdim;
+        const float lam = a.v_mix_lambda;
+        for (int e = lane; e < a.vdim; e += 32)
+          kv.v_pool[krow + (size_t)g * a.vdim + e] = fmaf(lam, first[e], (1.0f - lam) * pr[a.o_v + g * a.vdim + e]);
+        continue;
+      }
       for (int e = lane; e < a.vdim; e += 32) kv.v_pool[krow + (size_t)g * a.vdim + e] = pr[a.o_v + g * a.vdim + e];
       continue;
     }
@@ -313,13 +320,16 @@ __global__ void hyb_attn_prepare_kernel(tha_attn_t a, tha_rows_t rows, tha_kv_t 
     const float* cr = cos_t + (size_t)r * half;
     const float* sr = sin_t + (size_t)r * half;
     const float* wn = is_q ? a.q_norm : a.k_norm;   // per-channel weights sit inside the rotation, the row's factor outside
-    if (wn) wn += is_q ? h * a.dim : (h - a.heads) * a.dim;
+    if (wn && !a.head_norm) wn += is_q ? h * a.dim : (h - a.heads) * a.dim;
     float ss = 0.f;
-    if (a.unit_rms) {
+    if (a.head_norm) {
+      for (int d = lane; d < a.dim; d += 32) ss = fmaf(src[d], src[d], ss);
+      ss = warp_sum(ss);
+    } else if (a.unit_rms) {
       for (int d = lane; d < a.dim; d += 32) { const float v = hyb_rotated(src, d, rot_dims, a.rot_layout, cr, sr, wn); ss = fmaf(v, v, ss); }
       ss = warp_sum(ss);
     }
-    const float inv = (a.unit_rms ? 1.0f / sqrtf(ss / (float)a.dim + a.eps) : 1.0f) * (is_q ? q_mult * row_q : row_k);
+    const float inv = (a.unit_rms || a.head_norm ? 1.0f / sqrtf(ss / (float)a.dim + a.eps) : 1.0f) * (is_q ? q_mult * row_q : row_k);
     for (int d = lane; d < a.dim; d += 32) dst[d] = hyb_rotated(src, d, rot_dims, a.rot_layout, cr, sr, wn) * inv;
   }
 }
@@ -466,6 +476,7 @@ __global__ void __launch_bounds__(128) hyb_attn_kernel(tha_attn_t a, tha_rows_t 
       const bool vis = my_ok[rr] && hyb_attn_sees(a, t, my_pos[rr], my_first[rr]);
       float sv = vis ? sc[rr] * a.scale * my_scale[rr] : -INFINITY;
       if (a.softcap > 0.f && vis) sv = hyb_softcap(sv, a.softcap);
+      if (a.rel && vis) sv += hyb_attn_rel(a, g * gsize + part * AG + (warp * 4 + rr) % AG, my_pos[rr] - t);
       const float m_new = fmaxf(m_run[rr], warp_max(sv));
       float p = 0.f, corr = 1.f;
       if (m_new > -INFINITY) {
@@ -555,6 +566,8 @@ __global__ void __launch_bounds__(128) hyb_attn_kernel(tha_attn_t a, tha_rows_t 
 // keeps the online softmax of its rows among the four lanes that share a row, rounds the weights to bf16 (the row sums
 // add the rounded weights, so that they still sum to one) and multiplies them with V straight from the score registers:
 // two adjacent 8-key score tiles are one 16-deep A operand.  No exchange between warps; accumulators fp32.
+// With a distance bias (REL) the block's heads x the distances a tile can meet (its positions + 31) are staged beside the keys; a tile
+// that lies wholly where the bias no longer changes adds one register per row instead.
 // ------------------------------------------------------------------------------------------------------------------
 constexpr int AM_PAIRS = 64, AM_MAXD = 128;
 
@@ -569,7 +582,9 @@ __device__ __forceinline__ float attn_softcap_fast(float s, float cap, float two
   return cap - __fdividef(2.0f * cap, 1.0f + __expf(s * two_over_cap));
 }
 
-template <bool EXACT, bool CAP>
+__host__ __device__ inline int attn_rel_pitch(int AP) { return (AP + 31 - 8 + 31) / 32 * 32 + 8; }   // 8 banks from one head to the next
+
+template <bool EXACT, bool CAP, bool REL>
 __global__ void __launch_bounds__(128, 3) hyb_attn_mma_kernel(tha_attn_t a, tha_rows_t rows, tha_kv_t kv, const float* __restrict__ q,
                                                            __nv_bfloat16* __restrict__ out, int AG, int AP, int splits,
                                                            float* __restrict__ partial, const float* __restrict__ gate, long long ldg) {
@@ -579,6 +594,8 @@ __global__ void __launch_bounds__(128, 3) hyb_attn_mma_kernel(tha_attn_t a, tha_
   __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(smraw);   // [32][KS]
   __nv_bfloat16* Vs = Ks + ATT_KEYS * KS;                        // [32][VS], row-major like the cache: transposed on the way out
   const unsigned vs_base = (unsigned)__cvta_generic_to_shared(Vs);
+  float* Bs = REL ? reinterpret_cast<float*>(Vs + ATT_KEYS * VS) : nullptr;   // [AG][BP]: bias at distance (p_first - last key of the tile) + i
+  const int BP = REL ? attn_rel_pitch(AP) : 0;
   int seq = -1, r0 = 0, r_end = 0;
   {
     // the last tiles of a prompt see the most keys: they start first, so that the grid does not end on its longest blocks
@@ -625,6 +642,16 @@ __global__ void __launch_bounds__(128, 3) hyb_attn_mma_kernel(tha_attn_t a, tha_
     }
   }
   const float two_over_cap = CAP ? 2.0f / a.softcap : 0.f;
+  float row_far[2] = {0.f, 0.f};
+  const float* row_bias[2] = {Bs, Bs};   // this row's bias at key 0 of a tile; key i of the tile is i entries before it
+  if (REL) {
+#pragma unroll
+    for (int x = 0; x < 2; x++) {
+      const int pr = warp * 16 + lr + 8 * x;
+      if (row_ok[x]) row_far[x] = hyb_attn_rel(a, row_h[x], a.rel_n - 1);
+      row_bias[x] = Bs + (pr % AG) * BP + min(pr / AG, AP - 1) + ATT_KEYS - 1 - lc;
+    }
+  }
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   float oacc[AM_MAXD / 8][4];
 #pragma unroll
@@ -707,6 +734,14 @@ __global__ void __launch_bounds__(128, 3) hyb_attn_mma_kernel(tha_attn_t a, tha_
       }
     }
     }
+    const bool near = REL && p_first - (kt + ATT_KEYS - 1) < a.rel_n - 1;   // the same for the whole block
+    if (near) {
+      const int d0 = p_first - (kt + ATT_KEYS - 1);
+      for (int i = threadIdx.x; i < AG * (AP + ATT_KEYS - 1); i += blockDim.x) {
+        const int hl = i / (AP + ATT_KEYS - 1), n = i - hl * (AP + ATT_KEYS - 1), hg = part * AG + hl;
+        Bs[hl * BP + n] = hg < gsize ? hyb_attn_rel(a, g * gsize + hg, d0 + n) : 0.f;
+      }
+    }
     __syncthreads();
     // scores of this warp's 16 pairs against the 32 keys
     float sacc[4][4];
@@ -740,6 +775,7 @@ __global__ void __launch_bounds__(128, 3) hyb_attn_mma_kernel(tha_attn_t a, tha_
           const bool vis = row_ok[x] && hyb_attn_sees(a, t, row_pos[x], row_first[x]);
           float sv = sacc[j][2 * x + y] * a.scale * row_scale[x];
           if (CAP) sv = attn_softcap_fast(sv, a.softcap, two_over_cap);
+          if (REL) sv += near ? row_bias[x][-(8 * j + y)] : row_far[x];
           if (!vis) sv = -INFINITY;
           sacc[j][2 * x + y] = sv;
           mx = fmaxf(mx, sv);
@@ -1379,19 +1415,23 @@ __global__ void hyb_route_kernel(int experts, int top, int o_router, const float
 // Router with scores over ALL experts: s = softmax(z); the choice uses s + correction, limited to the `keep` groups (of
 // experts / groups neighbours each) whose largest choice score is highest -- experts outside them count as minus infinity,
 // whatever the sign of their score; the weights are the chosen s over their sum.  A warp per row; ties go to the lowest
-// index; needs top <= 32 and at most 4096 experts (blocks of 128 threads).
+// index; needs top <= 32 and at most 4096 experts (blocks of 128 threads).  SIGMOID: s = sigmoid(z), the weights are the chosen s times
+// `scale` and are not divided by their sum.
+template <bool SIGMOID>
 __global__ void hyb_route_groups_kernel(int experts, int top, int groups, int keep, int o_router, const float* __restrict__ correction,
                                         const float* __restrict__ proj, long long ldp, int n_rows, int* __restrict__ expert_id,
-                                        float* __restrict__ weight, int* __restrict__ counts) {
+                                        float* __restrict__ weight, int* __restrict__ counts, float scale) {
   const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (r >= n_rows) return;
   const float* z = proj + (size_t)r * ldp + o_router;
-  float zmax = -INFINITY;
-  for (int e = lane; e < experts; e += 32) zmax = fmaxf(zmax, z[e]);
-  for (int o = 16; o > 0; o >>= 1) zmax = fmaxf(zmax, __shfl_xor_sync(THA_FULL_MASK, zmax, o));
-  float den = 0.f;
-  for (int e = lane; e < experts; e += 32) den += expf(z[e] - zmax);
-  den = warp_sum(den);
+  float zmax = -INFINITY, den = 0.f;
+  if (!SIGMOID) {
+    for (int e = lane; e < experts; e += 32) zmax = fmaxf(zmax, z[e]);
+    for (int o = 16; o > 0; o >>= 1) zmax = fmaxf(zmax, __shfl_xor_sync(THA_FULL_MASK, zmax, o));
+    for (int e = lane; e < experts; e += 32) den += expf(z[e] - zmax);
+    den = warp_sum(den);
+  }
+  auto score = [&](int e) { return SIGMOID ? hyb_sigmoid(z[e]) : expf(z[e] - zmax) / den; };
   // bit g of the warp's words: group g may be chosen from (shared memory, so that any number of groups up to the experts fits)
   __shared__ unsigned allowed_s[4][128];
   unsigned* allowed = allowed_s[threadIdx.x >> 5];
@@ -1402,7 +1442,7 @@ __global__ void hyb_route_groups_kernel(int experts, int top, int groups, int ke
   if (bound) {
     auto group_best = [&](int g) {   // the largest choice score of group g
       float b = -INFINITY;
-      for (int e = g * per; e < (g + 1) * per; e++) b = fmaxf(b, expf(z[e] - zmax) / den + (correction ? correction[e] : 0.f));
+      for (int e = g * per; e < (g + 1) * per; e++) b = fmaxf(b, score(e) + (correction ? correction[e] : 0.f));
       return b;
     };
     const float gbest = lane < groups ? group_best(lane) : -INFINITY;   // lane g keeps group g's; groups beyond 32 are recomputed
@@ -1431,7 +1471,7 @@ __global__ void hyb_route_groups_kernel(int experts, int top, int groups, int ke
       const bool taken = n < 64 ? (taken_lo >> n) & 1ull : (taken_hi >> (n - 64)) & 1ull;
       const int g = groups > 1 ? e / per : 0;
       if (taken || !((allowed[g >> 5] >> (g & 31)) & 1u)) continue;
-      const float sc = expf(z[e] - zmax) / den;
+      const float sc = score(e);
       const float v = sc + (correction ? correction[e] : 0.f);
       if (v > best || (v == best && e < bi)) { best = v; bi = e; bs = sc; }
     }
@@ -1447,7 +1487,7 @@ __global__ void hyb_route_groups_kernel(int experts, int top, int groups, int ke
     if (lane == j) mine = bs;
     sum += bs;
   }
-  if (lane < top) weight[(size_t)r * top + lane] = mine / (sum + 1e-20f);
+  if (lane < top) weight[(size_t)r * top + lane] = SIGMOID ? mine * scale : mine / (sum + 1e-20f);
 }
 
 // any of the feed-forward activations (THA_ACT_*): gated ones read a gate value g and an up value u, ungated ones u only.
@@ -1737,12 +1777,14 @@ extern "C" int tha_hyb_attn_gated(void* stream, int dtype, const tha_attn_t* a, 
   if (a->v_share > 1 && (a->kv_heads % a->v_share || a->values_in_keys)) return THA_STATUS_INVALID_ARG;
   const int gsize = a->heads / a->kv_heads;
   // bf16 with heads the tensor-core form covers: 64 pairs per block; else 16 pairs on the fp32 cores
-  const bool tc = dtype == THA_DT_BF16 && hyb_tc_linear() && hyb_tc_attn() && a->dim % 16 == 0 && a->vdim % 8 == 0 && a->dim <= AM_MAXD && a->vdim <= AM_MAXD &&
+  if (a->rel && a->rel_n < 1) return THA_STATUS_INVALID_ARG;
+  const bool tc = !(a->rel && a->softcap > 0.f) && dtype == THA_DT_BF16 && hyb_tc_linear() && hyb_tc_attn() && a->dim % 16 == 0 && a->vdim % 8 == 0 && a->dim <= AM_MAXD && a->vdim <= AM_MAXD &&
                   (a->heads * a->vdim) % 2 == 0;
-  const bool wide = !tc && !gate && !a->head_scale && a->softcap <= 0.f && !a->out_f32 && a->v_share <= 1 && dtype == THA_DT_BF16 && hyb_tc_linear() && hyb_tc_attn() && hyb_attn_wide_ok(a);
+  const bool wide = !tc && !a->rel && !gate && !a->head_scale && a->softcap <= 0.f && !a->out_f32 && a->v_share <= 1 && dtype == THA_DT_BF16 && hyb_tc_linear() && hyb_tc_attn() && hyb_attn_wide_ok(a);
   const int pairs = wide ? hyb_attn_wide_pairs(a, rows) : tc ? AM_PAIRS : ATT_PAIRS;
   const int AG = gsize < pairs ? gsize : pairs, AP = pairs / AG;
-  const size_t smem = tc ? sizeof(__nv_bfloat16) * ((size_t)ATT_KEYS * (a->dim + 8) + (size_t)ATT_KEYS * (a->vdim + 8))
+  const size_t smem = tc ? sizeof(__nv_bfloat16) * ((size_t)ATT_KEYS * (a->dim + 8) + (size_t)ATT_KEYS * (a->vdim + 8)) +
+                               (a->rel ? sizeof(float) * (size_t)AG * attn_rel_pitch(AP) : 0)
                          : sizeof(float) * ((size_t)ATT_PAIRS * a->dim + (size_t)ATT_KEYS * (a->dim + 4) + (size_t)ATT_KEYS * a->vdim + ATT_PAIRS * ATT_KEYS);
   if (!wide && smem > 227 * 1024) return THA_STATUS_NOT_SUPPORTED;
   // position tiles: at most one ragged tile per sequence beyond rows / AP
@@ -1766,12 +1808,14 @@ extern "C" int tha_hyb_attn_gated(void* stream, int dtype, const tha_attn_t* a, 
       const int st = hyb_attn_wide_launch(s, a, rows, kv, q, (bf16*)out, grid, pairs, AG, AP, splits, split_scratch);
       if (st != THA_STATUS_SUCCESS) return st;
     } else if (tc) {
-      if (a->softcap > 0.f)
-        THA_CUDA_OK(launch(hyb_attn_mma_kernel<true, true>, grid, dim3(128), smem, s, false, *a, *rows, *kv, q, (bf16*)out, AG, AP, splits, split_scratch, gate, ldg));
+      if (a->rel)
+        THA_CUDA_OK(launch(hyb_attn_mma_kernel<true, false, true>, grid, dim3(128), smem, s, false, *a, *rows, *kv, q, (bf16*)out, AG, AP, splits, split_scratch, gate, ldg));
+      else if (a->softcap > 0.f)
+        THA_CUDA_OK(launch(hyb_attn_mma_kernel<true, true, false>, grid, dim3(128), smem, s, false, *a, *rows, *kv, q, (bf16*)out, AG, AP, splits, split_scratch, gate, ldg));
       else if (a->fp32_scores)
-        THA_CUDA_OK(launch(hyb_attn_mma_kernel<true, false>, grid, dim3(128), smem, s, false, *a, *rows, *kv, q, (bf16*)out, AG, AP, splits, split_scratch, gate, ldg));
+        THA_CUDA_OK(launch(hyb_attn_mma_kernel<true, false, false>, grid, dim3(128), smem, s, false, *a, *rows, *kv, q, (bf16*)out, AG, AP, splits, split_scratch, gate, ldg));
       else
-        THA_CUDA_OK(launch(hyb_attn_mma_kernel<false, false>, grid, dim3(128), smem, s, false, *a, *rows, *kv, q, (bf16*)out, AG, AP, splits, split_scratch, gate, ldg));
+        THA_CUDA_OK(launch(hyb_attn_mma_kernel<false, false, false>, grid, dim3(128), smem, s, false, *a, *rows, *kv, q, (bf16*)out, AG, AP, splits, split_scratch, gate, ldg));
     } else {
       if (a->vdim <= 256) {
         if (smem > 48 * 1024) THA_CUDA_OK(cudaFuncSetAttribute(hyb_attn_kernel<bf16, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
@@ -1919,11 +1963,13 @@ extern "C" int tha_hyb_moe_route(void* stream, const tha_moe_t* e, const float* 
   cudaStream_t s = (cudaStream_t)stream;
   int* counts = group_off + e->experts + 1;   // the second half of group_off is the routers' counters
   THA_CUDA_OK(cudaMemsetAsync(counts, 0, sizeof(int) * e->experts, s));
-  if (e->route == THA_ROUTE_SOFTMAX_GROUPS) {
+  if (e->route == THA_ROUTE_SOFTMAX_GROUPS || e->route == THA_ROUTE_SIGMOID_GROUPS) {
     const int groups = e->groups > 1 ? e->groups : 1;
     if (e->experts % groups || e->experts > 4096 || e->keep_groups < 1) return THA_STATUS_INVALID_ARG;
-    THA_CUDA_OK(launch(hyb_route_groups_kernel, dim3(ceil_div(n_rows, 4)), dim3(128), 0, s, false, e->experts, e->top, groups,
-                       e->keep_groups < groups ? e->keep_groups : groups, e->o_router, e->correction, proj, ldp, n_rows, expert_id, weight, counts));
+    auto kernel = e->route == THA_ROUTE_SIGMOID_GROUPS ? hyb_route_groups_kernel<true> : hyb_route_groups_kernel<false>;
+    THA_CUDA_OK(launch(kernel, dim3(ceil_div(n_rows, 4)), dim3(128), 0, s, false, e->experts, e->top, groups,
+                       e->keep_groups < groups ? e->keep_groups : groups, e->o_router, e->correction, proj, ldp, n_rows, expert_id, weight, counts,
+                       e->weight_scale));
   } else {
     THA_CUDA_OK(launch(hyb_route_kernel, dim3(ceil_div(n_rows, 4)), dim3(128), 0, s, false, e->experts, e->top, e->o_router, proj, ldp, n_rows,
                        expert_id, weight, counts));

@@ -11,6 +11,22 @@ __device__ __forceinline__ float hyb_load(const __nv_bfloat16* p) { return __bfl
 __device__ __forceinline__ void hyb_store(float* p, float v) { *p = v; }
 __device__ __forceinline__ void hyb_store(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 
+// V values at once (V = 4: 16-byte aligned fp32, 8-byte aligned bf16)
+__device__ __forceinline__ void hyb_load_vec(const float* p, float (&v)[1]) { v[0] = *p; }
+__device__ __forceinline__ void hyb_load_vec(const float* p, float (&v)[4]) {
+  const float4 t = *reinterpret_cast<const float4*>(p);
+  v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+}
+template <typename T>
+__device__ __forceinline__ void hyb_store_vec(T* p, const float (&v)[1]) { hyb_store(p, v[0]); }
+__device__ __forceinline__ void hyb_store_vec(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void hyb_store_vec(__nv_bfloat16* p, const float (&v)[4]) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+  uint2 t;
+  t.x = *reinterpret_cast<const unsigned*>(&lo); t.y = *reinterpret_cast<const unsigned*>(&hi);
+  *reinterpret_cast<uint2*>(p) = t;
+}
+
 __device__ __forceinline__ float hyb_softcap(float z, float cap) { return cap * tanhf(z / cap); }
 __device__ __forceinline__ float hyb_logsigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float hyb_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
@@ -46,6 +62,10 @@ __device__ __forceinline__ size_t hyb_kv_row(const tha_kv_t& kv, int slot, int t
 // Visibility of key t for a query at p whose block of positions starts at `first`:
 __device__ __forceinline__ bool hyb_attn_sees(const tha_attn_t& a, int t, int p, int first) {
   return t <= p && t >= first && (a.window <= 0 || p - t < a.window || t < a.keep_first);
+}
+// What the distance bias adds to head h's score of a key n positions back (a.rel given).
+__device__ __forceinline__ float hyb_attn_rel(const tha_attn_t& a, int h, int n) {
+  return __ldg(a.rel + (size_t)h * a.rel_n + min(max(n, 0), a.rel_n - 1));
 }
 // The key tiles (of 32, aligned to absolute multiples of 32) a block of queries at positions p_first..p_last walks: all from
 // the tile of key_lo to the tile of p_last, except, under a window, the run of tiles that lie wholly between the kept first

@@ -15,12 +15,12 @@
 namespace tha {
 
 // x = embed[token] * scale (+ the learned vector of the row's position when the model has a position table); x0, when given,
-// keeps a copy of it for the layers that add the embedding output again; join [rows, 2 width], when given, gets both halves of the
+// keeps a copy of it for the layers that add the embedding output again; copy (nullable) gets it in the products' number format; join [rows, 2 width], when given, gets both halves of the
 // joining map's input [x; embedding output] (the second half stays for the whole step)
 template <typename T>
 __global__ void hyb_embed_kernel(float* __restrict__ x, const T* __restrict__ embed, const int* __restrict__ token, int width,
                                  const T* __restrict__ pos_embed, const int* __restrict__ pos, float scale, float* __restrict__ x0,
-                                 T* __restrict__ join) {
+                                 T* __restrict__ copy, T* __restrict__ join) {
   const int r = blockIdx.x;
   const T* e = embed + (size_t)token[r] * width;
   const T* p = pos_embed ? pos_embed + (size_t)pos[r] * width : nullptr;
@@ -28,6 +28,7 @@ __global__ void hyb_embed_kernel(float* __restrict__ x, const T* __restrict__ em
     const float v = hyb_load(e + i) * scale + (p ? hyb_load(p + i) : 0.f);
     x[(size_t)r * width + i] = v;
     if (x0) x0[(size_t)r * width + i] = v;
+    if (copy) hyb_store(copy + (size_t)r * width + i, v);
     if (join) { hyb_store(join + (size_t)r * 2 * width + i, v); hyb_store(join + (size_t)r * 2 * width + width + i, v); }
   }
 }
@@ -118,6 +119,9 @@ static long long hyb_expert_rows() {
   return (v && *v) ? atoll(v) : 1024;
 }
 
+// row pitch of a stacked projection of n columns: rows start on 16-byte boundaries
+static int hyb_pitch(int n) { return (n + 3) / 4 * 4; }
+
 // channels of an attention layer's short convolution: its projected q | k | v columns (q alone when it reads another layer's rows,
 // q | k when the values are the keys)
 static size_t hyb_attn_conv_channels(const tha_attn_t& a) {
@@ -139,7 +143,7 @@ static size_t carve(const tha_hyb_model_t* m, const tha_rows_t* rows, int n_want
   };
   for (int i = 0; i < m->n_layers; i++) {
     const tha_hyb_layer_t& L = m->layers[i];
-    n_in = max(n_in, (size_t)L.n_in);
+    n_in = max(n_in, (size_t)hyb_pitch(L.n_in));
     if (L.block == THA_BLOCK_STREAMS) n_str = (size_t)(m->n_streams > 0 ? m->n_streams : 1);
     if (L.in_conv_taps > 0) hfw = W;
     if (L.pre_add_embed) keep_embed = true;
@@ -193,7 +197,7 @@ static size_t carve(const tha_hyb_model_t* m, const tha_rows_t* rows, int n_want
       av = max(av, (size_t)a.heads * a.kv_rank);
       mv = max(mv, (size_t)a.heads * a.vdim);
     }
-    if (L.has_norm2) { norm2 = true; n_in2 = max(n_in2, (size_t)L.n_in2); }
+    if (L.has_norm2) { norm2 = true; n_in2 = max(n_in2, (size_t)hyb_pitch(L.n_in2)); }
     if (L.has_ff == THA_FF_MOE) {
       top = max(top, (size_t)L.moe.top);
       ne = max(ne, (size_t)L.moe.experts);
@@ -330,15 +334,16 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
   carve(m, rows, n_want, sc.base, &b);
 
   const float embed_scale = m->embed_scale != 0.f ? m->embed_scale : 1.0f;
+  bool h_ready = false;   // what ran before already left this layer's first input in b.h (b.hf: see norm_out)
+  if (m->n_layers > 0 && m->layers[0].block == THA_BLOCK_POST) h_ready = true;   // the first mixer reads the embedding output itself
   if (dt == THA_DT_BF16)
     THA_CUDA_OK(launch(hyb_embed_kernel<bf16>, dim3(R), dim3(128), 0, s, false, b.x, (const bf16*)m->embed, rows->token, W, (const bf16*)m->pos_embed,
-                       rows->pos, embed_scale, b.x0, (bf16*)b.join));
+                       rows->pos, embed_scale, b.x0, h_ready ? (bf16*)b.h : (bf16*)nullptr, (bf16*)b.join));
   else
     THA_CUDA_OK(launch(hyb_embed_kernel<float>, dim3(R), dim3(128), 0, s, false, b.x, (const float*)m->embed, rows->token, W,
-                       (const float*)m->pos_embed, rows->pos, embed_scale, b.x0, (float*)b.join));
+                       (const float*)m->pos_embed, rows->pos, embed_scale, b.x0, h_ready ? (float*)b.h : (float*)nullptr, (float*)b.join));
   for (int i = 0; i < m->n_rot; i++) HYB_OK(tha_hyb_rotary_table(stream, &m->rot[i], rows->pos, R, b.cos_t[i], b.sin_t[i]));
 
-  bool h_ready = false;   // the previous block's last pass already left this layer's first norm in b.h (b.hf: see norm_out)
   bool join_ready = b.join != nullptr;   // the first half of b.join holds the current x
   // where a sequential layer's first norm goes, and in which format: a token-shifted mixer mixes it in fp32 first
   const tha_norm_t copy_x = {THA_NORM_COPY};
@@ -346,11 +351,12 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
   auto norm_dt = [&](const tha_hyb_layer_t& X) { return X.mixer == THA_MIX_WKV ? THA_DT_F32 : dt; };
   for (int li = 0; li < m->n_layers; li++) {
     const tha_hyb_layer_t& L = m->layers[li];
-    const long long ldp = L.n_in;
+    const long long ldp = hyb_pitch(L.n_in), ldp2 = hyb_pitch(L.n_in2);
     const bool seq = L.block == THA_BLOCK_SEQUENTIAL;
     const bool streams = L.block == THA_BLOCK_STREAMS;
+    const bool post = L.block == THA_BLOCK_POST;
     const int n_str = m->n_streams > 0 ? m->n_streams : 1;
-    const bool two_norms = !seq && !streams && L.has_norm2 && L.has_ff != THA_FF_NONE;
+    const bool two_norms = !seq && !streams && !post && L.has_norm2 && L.has_ff != THA_FF_NONE;
     if (streams) {
       // the mixer's input: the first sublayer's read of the streams and its norm (left behind by the previous layer's last
       // pass, or made here from the embedding output), then h + conv(h) continuing from the slot's tail
@@ -363,6 +369,10 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
         HYB_OK(tha_hyb_conv(stream, dt, rows, st, L.in_conv_state_off, b.hf, W, 0, W, L.in_conv_taps, L.in_conv_w, nullptr, 0, 1, 0, b.h));
         HYB_OK(tha_hyb_conv_tail(stream, rows, st, L.in_conv_state_off, b.hf, W, 0, W, L.in_conv_taps, nullptr));
       }
+    } else if (post) {   // the mixer reads x itself in the products' number format
+      if (!h_ready)
+        HYB_OK(tha_hyb_add_norm(stream, dt, b.x, nullptr, nullptr, 0.f, nullptr, 0.f, nullptr, nullptr, &copy_x, m->eps, b.h, 0, R, W));
+      h_ready = false;
     } else if (seq && h_ready) h_ready = false;
     else if (seq) {
       if (L.w_join) {   // x <- W_join [x; embedding output]
@@ -505,19 +515,19 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
         // the mixer's write and the feed-forward's read in one pass over the streams
         HYB_OK(tha_hyb_streams(stream, dt, b.xs, n_str, nullptr, &L.streams1, b.left, nullptr, 0, nullptr, nullptr, nullptr, nullptr, nullptr,
                                &L.streams2, &L.norm2, m->eps, 0, b.h2, R, W));
-        HYB_OK(tha_hyb_linear(stream, dt, b.proj2, L.n_in2, b.h2, W, 0, nullptr, L.w_in2, 0, R, L.n_in2, W, nullptr, 0));
+        HYB_OK(tha_hyb_linear(stream, dt, b.proj2, ldp2, b.h2, W, 0, nullptr, L.w_in2, 0, R, L.n_in2, W, nullptr, 0));
         if (L.has_ff == THA_FF_DENSE) {
           const tha_dense_ff_t& d = L.dense;
-          if (d.act == THA_ACT_POLYNORM) HYB_OK(tha_hyb_polynorm(stream, dt, b.sy, b.proj2, L.n_in2, d.o_up, d.b_up, d.act_c, m->eps, R, d.ff));
+          if (d.act == THA_ACT_POLYNORM) HYB_OK(tha_hyb_polynorm(stream, dt, b.sy, b.proj2, ldp2, d.o_up, d.b_up, d.act_c, m->eps, R, d.ff));
           else if (d.b_up) return THA_STATUS_NOT_SUPPORTED;
-          else HYB_OK(tha_hyb_ff_act(stream, dt, d.act, b.sy, b.proj2, L.n_in2, d.o_gate, d.o_up, R, d.ff, d.act_p, d.act_q));
+          else HYB_OK(tha_hyb_ff_act(stream, dt, d.act, b.sy, b.proj2, ldp2, d.o_gate, d.o_up, R, d.ff, d.act_p, d.act_q));
           HYB_OK(tha_hyb_linear(stream, dt, b.sdown, W, b.sy, d.ff, 0, nullptr, d.w_down, 0, R, W, d.ff, nullptr, 0));
           HYB_OK(tha_hyb_streams(stream, dt, b.xs, n_str, nullptr, &L.streams2, b.sdown, d.b_down, 0, nullptr, nullptr, nullptr, tap, sum_out,
                                  next ? &next->streams1 : nullptr, next ? &next->norm1 : nullptr, m->eps, nconv, nout, R, W));
         } else {
           const tha_moe_t& e = L.moe;
           if (e.shared_ff > 0) return THA_STATUS_NOT_SUPPORTED;
-          HYB_OK(hyb_run_experts(stream, sc, dt, R, W, e, b.h2, b.proj2, L.n_in2, b));
+          HYB_OK(hyb_run_experts(stream, sc, dt, R, W, e, b.h2, b.proj2, ldp2, b));
           HYB_OK(tha_hyb_streams(stream, dt, b.xs, n_str, nullptr, &L.streams2, nullptr, nullptr, e.top, b.weight, b.inv, b.down, tap, sum_out,
                                  next ? &next->streams1 : nullptr, next ? &next->norm1 : nullptr, m->eps, nconv, nout, R, W));
         }
@@ -537,8 +547,8 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
       if (L.has_ff == THA_FF_DENSE) {
         const tha_dense_ff_t& d = L.dense;
         HYB_OK(tha_hyb_add_norm(stream, dt, b.x, b.left, left_b, cl, right, cr, nullptr, nullptr, &L.norm2, m->eps, b.h2, 0, R, W));
-        HYB_OK(tha_hyb_linear(stream, dt, b.proj2, L.n_in2, b.h2, W, 0, nullptr, L.w_in2, 0, R, L.n_in2, W, nullptr, 0));
-        HYB_OK(tha_hyb_ff_act(stream, dt, d.act, b.sy, b.proj2, L.n_in2, d.o_gate, d.o_up, R, d.ff, d.act_p, d.act_q));
+        HYB_OK(tha_hyb_linear(stream, dt, b.proj2, ldp2, b.h2, W, 0, nullptr, L.w_in2, 0, R, L.n_in2, W, nullptr, 0));
+        HYB_OK(tha_hyb_ff_act(stream, dt, d.act, b.sy, b.proj2, ldp2, d.o_gate, d.o_up, R, d.ff, d.act_p, d.act_q));
         HYB_OK(tha_hyb_linear(stream, dt, b.sdown, W, b.sy, d.ff, 0, nullptr, d.w_down, 0, R, W, d.ff, nullptr, 0));
         ffo = b.sdown;
       } else if (L.has_ff == THA_FF_NONE && !right) {
@@ -574,20 +584,55 @@ extern "C" int tha_hyb_step(void* stream, const tha_hyb_model_t* m, const tha_ro
       h_ready = next != nullptr;
       continue;
     }
+    if (post) {
+      // x += m norm1(mixer) with a copy for the feed-forward's product; then x += m norm2(ff), the tap and a copy for the next mixer: each
+      // one pass over x, the second one also puts the feed-forward's parts together
+      const tha_hyb_layer_t* next = li + 1 < m->n_layers && m->layers[li + 1].block == THA_BLOCK_POST ? &m->layers[li + 1] : nullptr;
+      float* tap = taps ? taps + (size_t)li * R * W : (float*)nullptr;
+      void* hand_on = next ? b.h : nullptr;
+      const bool ff = L.has_ff != THA_FF_NONE;
+      HYB_OK(tha_hyb_post_norm(stream, dt, b.x, b.left, nullptr, 0, 0, nullptr, nullptr, nullptr, L.res_mult, &L.norm1, m->eps, ff ? nullptr : tap,
+                               ff ? b.h : hand_on, R, W));
+      if (ff) {
+        HYB_OK(tha_hyb_linear(stream, dt, b.proj2, ldp2, b.h, W, 0, nullptr, L.w_in2, 0, R, L.n_in2, W, nullptr, 0));
+        const float* dense = nullptr;
+        const float* dense_gate = nullptr;
+        int top = 0;
+        if (L.has_ff == THA_FF_DENSE) {
+          const tha_dense_ff_t& d = L.dense;
+          HYB_OK(tha_hyb_ff_act(stream, dt, d.act, b.sy, b.proj2, ldp2, d.o_gate, d.o_up, R, d.ff, d.act_p, d.act_q));
+          HYB_OK(tha_hyb_linear(stream, dt, b.sdown, W, b.sy, d.ff, 0, nullptr, d.w_down, 0, R, W, d.ff, nullptr, 0));
+          dense = b.sdown;
+        } else {
+          const tha_moe_t& e = L.moe;
+          top = e.top;
+          HYB_OK(hyb_run_experts(stream, sc, dt, R, W, e, b.h, b.proj2, ldp2, b));
+          if (e.shared_ff > 0) {
+            HYB_OK(tha_hyb_ff_act(stream, dt, e.act, b.sy, b.proj2, ldp2, e.o_sgate, e.o_sup, R, e.shared_ff, e.shared_limit, e.alpha));
+            HYB_OK(tha_hyb_linear(stream, dt, b.sdown, W, b.sy, e.shared_ff, 0, nullptr, e.w_sdown, 0, R, W, e.shared_ff, nullptr, 0));
+            dense = b.sdown;
+            if (e.shared_scaled) dense_gate = b.proj2 + e.o_sscale;
+          }
+        }
+        HYB_OK(tha_hyb_post_norm(stream, dt, b.x, dense, dense_gate, ldp2, top, b.weight, b.inv, b.down, L.res_mult, &L.norm2, m->eps, tap, hand_on, R, W));
+      }
+      h_ready = next != nullptr;
+      continue;
+    }
     // the feed-forward reads the mixer's normed input, or a second norm of the same x through its own stacked product
     const void* hf = b.h;
     const float* fproj = b.proj;
     long long ldf = ldp;
     if (two_norms) {
-      HYB_OK(tha_hyb_linear(stream, dt, b.proj2, L.n_in2, b.h2, W, 0, nullptr, L.w_in2, 0, R, L.n_in2, W, nullptr, 0));
-      hf = b.h2; fproj = b.proj2; ldf = L.n_in2;
+      HYB_OK(tha_hyb_linear(stream, dt, b.proj2, ldp2, b.h2, W, 0, nullptr, L.w_in2, 0, R, L.n_in2, W, nullptr, 0));
+      hf = b.h2; fproj = b.proj2; ldf = ldp2;
     }
     int top = 0;
     const float* sdown = nullptr;
     const float* sgate = nullptr;
     if (L.has_ff == THA_FF_DENSE) {
       const tha_dense_ff_t& d = L.dense;
-      HYB_OK(tha_hyb_ff_act(stream, dt, d.act, b.sy, fproj, ldf, d.o_gate, d.o_up, R, d.ff, 0.f, 0.f));
+      HYB_OK(tha_hyb_ff_act(stream, dt, d.act, b.sy, fproj, ldf, d.o_gate, d.o_up, R, d.ff, d.act_p, d.act_q));
       HYB_OK(tha_hyb_linear(stream, dt, b.sdown, W, b.sy, d.ff, 0, nullptr, d.w_down, 0, R, W, d.ff, nullptr, 0));
       sdown = b.sdown;
     } else if (L.has_ff == THA_FF_MOE) {

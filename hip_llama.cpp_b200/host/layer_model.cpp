@@ -19,6 +19,7 @@ void register_numizen();   // host/arch_numizen.cpp
 void register_bozovik();   // host/arch_bozovik.cpp
 void register_mozetar();   // host/arch_mozetar.cpp
 void register_logulix();   // host/arch_logulix.cpp
+void register_gavodra();   // host/arch_gavodra.cpp
 
 // ---- registry -----------------------------------------------------------------------------------------------------
 static std::vector<ArchitectureEntry>& registry() {
@@ -34,6 +35,7 @@ static void register_builtin() {
     register_bozovik();
     register_mozetar();
     register_logulix();
+    register_gavodra();
   });
 }
 void register_architecture(const ArchitectureEntry& e) {
@@ -212,6 +214,19 @@ struct Stack {
 };
 }  // namespace
 
+// The distance buckets of AttnSpec::rel written out: row of the table for every distance up to the first that reads the last row.
+// rows / 2 + floor(ln(n / half) / ln(far / half) * (rows - half)); the small addend keeps distances that lie exactly on a step on it.
+static std::vector<int> distance_rows(int rows, double far) {
+  const int half = rows / 2, last = rows - 1;
+  std::vector<int> of;
+  for (int n = 0; of.empty() || of.back() != last; n++) {
+    if (n < half) { of.push_back(n); continue; }
+    const double step = floor(log((double)n / half) / log(far / half) * (rows - half) + 1e-9);
+    of.push_back((int)fmin((double)last, half + step));
+  }
+  return of;
+}
+
 LayerModel* LayerModel::load(const std::string& folder, int dtype, std::string* err) {
   JsonValue config;
   const ArchitectureEntry* e = detect_model(folder, &config, err);
@@ -328,7 +343,7 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
       A.heads = a.heads * maps; A.kv_heads = a.kv_heads * maps;
       const long long cq = (long long)A.heads * a.dim, ck = (long long)A.kv_heads * a.dim, cv = (long long)a.kv_heads * a.vdim;
       if (a.v_is_k && (a.vdim != a.dim || a.diff || a.kv_from >= 0)) throw std::runtime_error("attention: values that are the keys need vdim == dim, one map per head and rows of their own");
-      if ((!a.q_norm.empty() || !a.k_norm.empty()) && a.diff) throw std::runtime_error("attention: row norms of differential projections are not served");
+      if ((!a.q_norm.empty() || !a.k_norm.empty() || a.head_norm) && a.diff) throw std::runtime_error("attention: row norms of differential projections are not served");
       if (a.softcap < 0.f) throw std::runtime_error("attention: the score cap must be positive");
       m->separate_values_ = true;
       if (a.kv_from >= 0) {
@@ -372,8 +387,35 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
         else A.o_v = in.add(a.v, cv);
       }
       A.softcap = a.softcap;
-      if (!a.q_norm.empty()) A.q_norm = vec(a.q_norm, (size_t)cq);
-      if (!a.k_norm.empty() && a.kv_from < 0) A.k_norm = vec(a.k_norm, (size_t)ck);
+      A.head_norm = a.head_norm;
+      if (!a.q_norm.empty()) A.q_norm = vec(a.q_norm, (size_t)(a.head_norm ? a.dim : cq));
+      if (!a.k_norm.empty() && a.kv_from < 0) A.k_norm = vec(a.k_norm, (size_t)(a.head_norm ? a.dim : ck));
+      if (!a.rel.empty()) {
+        const TensorInfo& t = file.info(a.rel);
+        if (t.shape.size() != 2 || t.shape[0] < 2 || t.shape[1] != A.heads) throw std::runtime_error("tensor '" + a.rel + "': a distance table is [rows, heads] with at least two rows");
+        const int rows = (int)t.shape[0];
+        if (!(a.rel_far > rows / 2) || a.rel_far > (double)(1 << 20))
+          throw std::runtime_error("attention: the distance at which the bias table ends must lie beyond half of its rows (and within 2^20)");
+        std::vector<float> tab, full;
+        file.read_f32(a.rel, &tab);
+        const std::vector<int> of = distance_rows(rows, a.rel_far);
+        for (int h = 0; h < A.heads; h++)
+          for (int row : of) full.push_back(tab[(size_t)row * A.heads + h]);
+        A.rel = (const float*)m->upload(full.data(), full.size() * 4);
+        A.rel_n = (int)of.size();
+      }
+      if (a.v_mix_from >= 0) {
+        if ((size_t)a.v_mix_from >= li_now || a.kv_from >= 0 || a.v_is_k || a.conv_taps > 0) throw std::runtime_error("attention: value mixing needs an earlier layer and values of its own");
+        const LayerSpec& d = spec.layers[a.v_mix_from];
+        if (d.mixer != THA_MIX_ATTN || d.same_weights_as >= 0 || d.attn.kv_from >= 0 || (long long)d.attn.kv_heads * d.attn.vdim != cv)
+          throw std::runtime_error("attention: value mixing needs an earlier attention layer with as many value channels");
+        std::vector<float> lam;
+        file.read_f32(a.v_mix, &lam);
+        if (lam.size() != 1) throw std::runtime_error("tensor '" + a.v_mix + "' must be one number");
+        A.v_mix = 1;
+        A.v_mix_layer = m->layers_[a.v_mix_from].attn.cache_layer;
+        A.v_mix_lambda = lam[0];
+      }
       if (!a.o_b.empty()) A.b_o = vec(a.o_b, W);
       A.q_temp_coef = a.q_temp_coef; A.q_temp_every = a.q_temp_every > 0 ? a.q_temp_every : 0;
       const bool biased = !a.q_b.empty() || !a.k_b.empty();
@@ -453,6 +495,8 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
         L.w_join = join_matrix(ls.pre_join);
         if ((L.mixer == THA_MIX_ATTN || L.mixer == THA_MIX_ATTN_GDELTA) && L.attn.kv_shared)
           throw std::runtime_error("a repeated attention layer with another layer's cache rows is not served");
+        if ((L.mixer == THA_MIX_ATTN || L.mixer == THA_MIX_ATTN_GDELTA) && L.attn.v_mix)
+          throw std::runtime_error("a repeated attention layer with value mixing is not served");
         if ((L.mixer == THA_MIX_ATTN || L.mixer == THA_MIX_ATTN_GDELTA) && L.attn.conv_taps > 0) {
           const tha_attn_t& A = L.attn;
           const long long C = (long long)A.heads * A.dim + (long long)A.kv_heads * A.dim +
@@ -507,6 +551,10 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
         throw std::runtime_error("a joining map, an output bias and token-shifted mixers are served in sequential blocks");
       if (ls.block == THA_BLOCK_SEQUENTIAL && ls.has_ff && (ls.ff_kind != THA_FF_DENSE || ls.norm2.empty()))
         throw std::runtime_error("a sequential block serves a dense feed-forward behind a second norm, or none");
+      if (ls.block == THA_BLOCK_POST && (spec.norm_kind != THA_NORM_RMS || (ls.has_ff && ls.norm2.empty()) || ls.mixer == THA_MIX_PARALLEL ||
+                                         ls.mixer == THA_MIX_ATTN_GDELTA || ls.side.dim > 0 || ls.pre_add_embed || !ls.pre_vec.empty() || !ls.scale_mix.empty() ||
+                                         !ls.scale_ff.empty()))
+        throw std::runtime_error("a post-norm block serves one-sided mixers and rms norms, one for each sublayer, and nothing ahead of them");
       L.norm1 = norm(ls.norm1);
       if (ls.block == THA_BLOCK_STREAMS) {
         const int n = spec.n_streams;
@@ -787,6 +835,7 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
           if (c.size() != 4) throw std::runtime_error("tensor '" + d.act_params + "' must hold four numbers");
           for (int i = 0; i < 4; i++) L.dense.act_c[i] = c[i];
         }
+        if (d.act == THA_ACT_GLU_CLAMPED) { L.dense.act_p = d.limit; L.dense.act_q = d.alpha; }
         if (d.act == THA_ACT_XIELU) {
           std::vector<float> pq;
           file.read_f32(d.act_params, &pq);
@@ -799,7 +848,8 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
         tha_moe_t& E = L.moe;
         E.experts = e.experts; E.top = e.top; E.ff = e.ff; E.limit = e.limit; E.alpha = e.alpha;
         E.act = e.act; E.route = e.route;
-        if (e.route == THA_ROUTE_SOFTMAX_GROUPS) {
+        E.weight_scale = e.weight_scale;
+        if (e.route == THA_ROUTE_SOFTMAX_GROUPS || e.route == THA_ROUTE_SIGMOID_GROUPS) {
           const int groups = e.groups > 1 ? e.groups : 1, keep = e.groups > 1 ? e.keep_groups : 1;
           if (e.experts % groups || keep < 1 || keep > groups || e.experts > 4096)
             throw std::runtime_error("mixture of experts: groups must divide the experts (at most 4096 experts), 1 <= keep <= groups");
@@ -878,7 +928,7 @@ LayerModel* LayerModel::build(const LayerProgramSpec& spec, const SafeTensors& f
         M.final_norm.b = (const float*)m->upload(b.data(), b.size() * 4);
       }
     }
-    M.head = mat(spec.head, spec.vocab, W);
+    M.head = spec.head == spec.embed ? M.embed : mat(spec.head, spec.vocab, W);
     M.layers = m->layers_.data();
     M.n_rot = (int)m->rot_.size();
     M.rot = m->rot_.data();

@@ -30,6 +30,10 @@ class JsonValue {
     return num;
   }
   int integer() const { return (int)number(); }
+  bool boolean() const {
+    if (kind != Bool) throw std::runtime_error("config: true or false was expected");
+    return b;
+  }
   const std::string& string() const {
     if (kind != String) throw std::runtime_error("config: a string was expected");
     return str;

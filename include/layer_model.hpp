@@ -58,6 +58,13 @@ struct AttnSpec {
   std::string q_norm, k_norm;            // rms norms over the whole q row [heads * dim] and k row [kv_heads * dim]; empty: none
   bool v_is_k = false;                   // no value tensor: values are the convolved keys, not normed or rotated
   float softcap = 0.f;                   // > 0: scores s become softcap * tanh(s / softcap)
+  bool head_norm = false;                // q_norm / k_norm are [dim], applied to every head divided by its own root mean square
+  // a learned bias per head by distance bucket [rows, heads]; empty: none.  Distances below rows / 2 have a row each, the rest share the
+  // other rows in logarithmic steps that end at rel_far
+  std::string rel;
+  double rel_far = 0.0;
+  int v_mix_from = -1;                   // >= 0: values become (1 - lambda) v + lambda v', v' the values of that earlier layer (index into `layers`)
+  std::string v_mix;                     // lambda: one number
   int kv_from = -1;                      // >= 0: no key / value tensors; the layer reads the cache rows of that layer (index into `layers`)
 };
 struct HgrnSpec {
@@ -114,6 +121,7 @@ struct LatentSpec {
 struct DenseSpec {
   int ff = 0, act = THA_ACT_GELU_TANH_GLU;
   std::string gate, up, down;            // ungated activations have no `gate`
+  float limit = 0.f, alpha = 1.702f;     // THA_ACT_GLU_CLAMPED
   std::string act_params;                // THA_ACT_XIELU: [2]; THA_ACT_POLYNORM: [4]
   std::string up_b, down_b;              // biases; empty: none
 };
@@ -123,7 +131,8 @@ struct MoeSpec {
   std::string router, prefix;            // expert e's tensors: prefix + "e<e>.gate" / ".up" / ".down" (ungated: no ".gate")
   std::string s_gate, s_up, s_down;
   int act = THA_ACT_GLU_CLAMPED, route = THA_ROUTE_TOPK_SOFTMAX;
-  std::string correction;                // THA_ROUTE_SOFTMAX_GROUPS
+  std::string correction;                // THA_ROUTE_*_GROUPS
+  float weight_scale = 1.0f;             // THA_ROUTE_SIGMOID_GROUPS
   int groups = 0, keep_groups = 0;
   std::string s_scale;                   // [1, width]: the shared expert is multiplied by sigmoid of this product; empty: none
 };
@@ -144,7 +153,7 @@ struct LayerSpec {
   std::string left_out, right_out;
   DeltaSpec delta;
   int block = THA_BLOCK_PARALLEL;
-  float res_mult = 1.0f;                 // sequential blocks
+  float res_mult = 1.0f;                 // sequential and post-norm blocks
   GDeltaSpec gdelta;                     // THA_MIX_ATTN_GDELTA (beside attn)
   float mix_left = 1.0f, mix_right = 1.0f;
   SideSpec side;

@@ -43,6 +43,7 @@ extern "C" {
 #define THA_BLOCK_PARALLEL 0   /* x <- x + mixer(norm1 x) + ff(norm x): mixer and feed-forward read the same x */
 #define THA_BLOCK_SEQUENTIAL 1 /* x <- x + m mixer(norm1 x), then x <- x + m ff(norm2 x), then the per-token side input */
 #define THA_BLOCK_STREAMS 2    /* several residual streams: every sublayer reads a weighted sum of them and writes to all (tha_streams_t) */
+#define THA_BLOCK_POST 3       /* x <- x + m norm1(mixer(x)), x <- x + m norm2(ff(x)): the sublayers read x itself, rms norms weigh what they return */
 
 #define THA_NORM_RMS 0     /* x / sqrt(mean(x^2) + eps) * (w_offset + w) */
 #define THA_NORM_DYT 1     /* tanh(alpha * x) * w + b: element-wise, no statistics */
@@ -64,6 +65,8 @@ extern "C" {
 #define THA_ROUTE_TOPK_SOFTMAX 0    /* the top logits, softmax over the chosen */
 #define THA_ROUTE_SOFTMAX_GROUPS 1  /* softmax over all experts; choice by score + correction inside the best groups of
                                        neighbouring experts; weights = the chosen scores (uncorrected) over their sum */
+#define THA_ROUTE_SIGMOID_GROUPS 2  /* the same choice (correction, groups) on sigmoid scores; weights = the chosen scores
+                                       (uncorrected) times weight_scale, not divided by their sum */
 
 #define THA_GATE_SIGMOID 0
 #define THA_GATE_SILU 1
@@ -171,6 +174,15 @@ typedef struct {
   const float* k_norm;     /* [kv_heads * dim] */
   float softcap;           /* > 0: a scaled score s becomes softcap * tanh(s / softcap) ahead of the softmax */
   const float* b_o;        /* [width] bias of the output projection (sequential blocks), NULL: none */
+  int head_norm;           /* 1: every q and k head is divided by its own root mean square over dim ahead of rotation; q_norm and k_norm
+                              are then [dim], shared by the heads (NULL: no weight) */
+  /* distance bias (NULL: none): head h's scaled (and capped) score of a key n = p - j positions back gets rel[h * rel_n + min(n, rel_n - 1)] */
+  const float* rel;        /* [heads, rel_n] */
+  int rel_n;
+  /* value mixing (v_mix 1): the cached value row is (1 - v_mix_lambda) v + v_mix_lambda v', v' the value row that cache layer v_mix_layer
+   * (an earlier layer of the step, as many value channels) holds for the same token */
+  int v_mix, v_mix_layer;
+  float v_mix_lambda;
 } tha_attn_t;
 
 /* Generalized delta rule with a decay and a removal rate per key channel.  r, k, v, g: heads x dim columns each.
@@ -325,7 +337,7 @@ typedef struct {
   int ff, act;
   int o_gate, o_up;     /* columns of the feed-forward's stacked input projection (ungated activations: o_up only) */
   const void* w_down;   /* [width, ff] */
-  float act_p, act_q;   /* THA_ACT_XIELU: the two stored numbers (softplus is taken by the kernel) */
+  float act_p, act_q;   /* THA_ACT_XIELU: the two stored numbers (softplus is taken by the kernel); THA_ACT_GLU_CLAMPED: limit, alpha */
   /* zero-initialised, the fields below keep the behaviour described above */
   const float* b_up;    /* [ff] added to W_up h before the activation, NULL: none */
   const float* b_down;  /* [width] added to the result, NULL: none */
@@ -356,10 +368,11 @@ typedef struct {
   /* zero-initialised, the fields below keep the behaviour described above */
   int act;               /* THA_ACT_*; ungated activations: w_gate_up is [experts][ff, width] (up rows only) */
   int route;             /* THA_ROUTE_* */
-  const float* correction; /* [experts], THA_ROUTE_SOFTMAX_GROUPS: added to the scores for the choice only */
+  const float* correction; /* [experts], THA_ROUTE_*_GROUPS: added to the scores for the choice only */
   int groups, keep_groups; /* groups <= 1: every expert can be chosen */
   int shared_scaled;     /* 1: the shared expert's output is multiplied by sigmoid of column o_sscale (one number per row) */
   int o_sscale;
+  float weight_scale;    /* THA_ROUTE_SIGMOID_GROUPS */
 } tha_moe_t;
 
 typedef struct {
@@ -387,7 +400,7 @@ typedef struct {
   tha_dense_ff_t dense; /* THA_FF_DENSE */
   /* zero-initialised, the fields below keep the behaviour described above */
   int block;            /* THA_BLOCK_*; sequential blocks: dense or no feed-forward, reading norm2 through w_in2 */
-  float res_mult;       /* THA_BLOCK_SEQUENTIAL: m */
+  float res_mult;       /* THA_BLOCK_SEQUENTIAL, THA_BLOCK_POST: m (post-norm blocks: any feed-forward through w_in2, norm1 and norm2 on the results) */
   tha_gdelta_t gdelta;  /* THA_MIX_ATTN_GDELTA (beside attn) */
   float mix_left, mix_right; /* THA_MIX_ATTN_GDELTA */
   tha_side_t side;
@@ -485,6 +498,12 @@ int tha_hyb_side_gate(void* stream, int dtype, void* out, const float* gate_raw,
 int tha_hyb_block_finish(void* stream, int dtype, float* x, const float* ff, const float* ff_b, const float* y, float m, const float* y_norm, float eps,
                          float* tap, const float* embed_out, const float* vec, const tha_norm_t* next_norm, void* out, long long ldo,
                          int n_rows, int width);
+/* the end of a post-norm sublayer, one pass over x: y = dense * sigmoid(dense_gate[r * ldg]) + sum_j weight[r, j] * down[inv[r, j]] (dense
+ * [n_rows, width], NULL: none; dense_gate NULL: factor 1; top picks of a mixture, top 0: none); x += m * y / sqrt(mean(y^2) + eps) *
+ * (norm->w_offset + norm->w); tap (nullable) receives x; out (nullable) x in the products' number format */
+int tha_hyb_post_norm(void* stream, int dtype, float* x, const float* dense, const float* dense_gate, long long ldg, int top,
+                      const float* weight, const int* inv, const float* down, float m, const tha_norm_t* norm, float eps, float* tap,
+                      void* out, int n_rows, int width);
 /* x += c_left * (left + left_b) + c_right * right (left_b, right NULL: none) (+ embed_out when given) (+ vec when given); then, with n not NULL,
  * out (dtype-typed, row pitch ldo; 0: width) = the norm n of x (THA_NORM_COPY: x itself).  left NULL: only the optional addends. */
 int tha_hyb_add_norm(void* stream, int dtype, float* x, const float* left, const float* left_b, float c_left, const float* right,
