@@ -516,3 +516,60 @@ def random_logulix_tensors(cfg: dict, seed: int = 0, decay_rank: int = 16) -> di
             a = 1.0 + 0.2 * rng.standard_normal(shape)
         out[name] = np.asarray(a, dtype=np.float32)
     return out
+
+
+def gavodra_tensor_shapes(cfg: dict, rel_rows: int = 32) -> dict:
+    """name -> shape of every tensor a Gavodra config asks for (rel_rows: rows of the distance tables, a property of the tensors
+    and not of the config)."""
+    W, V = cfg["width"], cfg["vocab"]
+    s = {"embed": (V, W), "final.norm": (W,)}
+
+    def glu(q, ff):
+        s[q + "gate"], s[q + "up"], s[q + "down"] = (ff, W), (ff, W), (W, ff)
+
+    for i, L in enumerate(cfg["layers"]):
+        p, m, q = f"l{i}.", L["mixer"], f"l{i}.mix."
+        if L["type"] != "attention":
+            raise ValueError(L["type"])
+        H, G, D, E = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        s[p + "norm1"] = (W,)
+        s[q + "q"], s[q + "k"], s[q + "v"], s[q + "g"], s[q + "o"] = (H * D, W), (G * D, W), (G * E, W), (H, W), (W, H * E)
+        s[q + "q.norm"], s[q + "k.norm"], s[q + "rel"] = (D,), (D,), (rel_rows, H)
+        if m.get("v_mix"):
+            s[q + "vmix"] = ()
+        f = L.get("mlp")
+        if not f:
+            continue
+        s[p + "norm2"] = (W,)
+        q = p + "mlp."
+        if f["kind"] == "dense":
+            glu(q, f["ff"])
+        else:
+            s[q + "router"], s[q + "correction"] = (f["router"]["experts"], W), (f["router"]["experts"],)
+            for e in range(f["router"]["experts"]):
+                glu(q + f"e{e}.", f["expert"]["ff"])
+            if f.get("shared"):
+                glu(q + "shared.", f["shared"]["ff"])
+                s[q + "shared.sg"] = (1, W)
+    return s
+
+
+def random_gavodra_tensors(cfg: dict, seed: int = 0, rel_rows: int = 32) -> dict:
+    """Random weights of a Gavodra config: matrices N(0, 1/in), norm weights around one, distance biases of order one half, value
+    mixing shares in (0.2, 0.8), small choice corrections."""
+    rng = np.random.default_rng(seed)
+    out = {}
+    for name, shape in gavodra_tensor_shapes(cfg, rel_rows).items():
+        last = name.rsplit(".", 1)[-1]
+        if last == "rel":
+            a = 0.5 * rng.standard_normal(shape)
+        elif last == "vmix":
+            a = rng.uniform(0.2, 0.8)
+        elif last == "correction":
+            a = 0.1 * rng.standard_normal(shape)
+        elif len(shape) == 2:
+            a = rng.standard_normal(shape, dtype=np.float32) * (1.0 if name == "embed" else 1.0 / np.sqrt(shape[1]))
+        else:
+            a = 1.0 + 0.2 * rng.standard_normal(shape)
+        out[name] = np.asarray(a, dtype=np.float32)
+    return out

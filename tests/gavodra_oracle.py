@@ -6,7 +6,9 @@ portions and single tokens alike.
 
 A layer norms what a sublayer returns, not what it reads:  x <- x + m N1(mixer(x)),  x <- x + m N2(ff(x)).
 """
+import functools
 import math
+from fractions import Fraction
 
 import numpy as np
 
@@ -20,13 +22,14 @@ def rms_unit(x, eps):
 
 
 # ---- the distance bias ----------------------------------------------------------------------------------------------------
+@functools.lru_cache(maxsize=None)
 def bucket(n, rows, far):
     """Which of `rows` table rows the distance n >= 0 reads: its own below rows / 2, then logarithmically wider ones that end at `far`.
     Whole-number comparison: step k of the upper half starts where (n / half)^steps >= (far / half)^k."""
     half = rows // 2
     if n < half:
         return n
-    steps, far = rows - half, int(far)
+    steps, far = rows - half, Fraction(far)
     k = 0
     while k + 1 < steps and n ** steps * half ** (k + 1) >= far ** (k + 1) * half ** steps:
         k += 1

@@ -9,6 +9,7 @@ import numpy as np
 import pytest
 
 import bozovik_oracle as B
+import gavodra_oracle as G
 import logulix_oracle as L
 import mozetar_oracle as M
 import numizen_oracle as N
@@ -44,7 +45,7 @@ def test_registry_names_what_it_knows(tmp_path):
     with pytest.raises(serving.ServingError) as e:
         serving.ServingEngine(str(tmp_path), "float32", 64, 1)
     assert "Nope" in str(e.value) and "Timerax" in str(e.value) and "llama2" in str(e.value) and "Numizen" in str(e.value)
-    assert "Bozovik" in str(e.value) and "Mozetar" in str(e.value) and "Logulix" in str(e.value)
+    assert "Bozovik" in str(e.value) and "Mozetar" in str(e.value) and "Logulix" in str(e.value) and "Gavodra" in str(e.value)
 
 
 @built
@@ -424,3 +425,80 @@ def test_plain_logulix_runs_bonus_and_values():
          "q.norm": np.ones(4), "k.norm": np.ones(2), "o": np.eye(4)[:2], "o.b": np.array([0.5, 0.0])}
     y = L.attention_mixer(np.array([[1.0, 2.0], [3.0, 4.0]]), m, {"p." + k: v for k, v in W.items()}, "p.", 1e-6, {}, 0)
     assert np.allclose(y, [[2.0 + 0.5, 2.0], [20.0 + 4.0 + 0.5, 20.0 + 4.0]])
+
+
+# ---- Gavodra ----------------------------------------------------------------------------------------------------------
+GAVODRA_MIXER = {"heads": 4, "kv_heads": 2, "dim": 6, "vdim": 5, "scale": 0.4, "bias_max": 30, "v_mix": True}
+GAVODRA_MOE = {"kind": "moe", "expert": {"ff": 7, "limit": 0.9}, "router": {"experts": 3, "top": 2, "scale": 1.5}, "shared": {"ff": 8, "limit": 0.7}}
+
+
+def _gavodra_cfg(layers, **extra):
+    c = {"architecture": "Gavodra", "width": 16, "vocab": 20, "norm": {"eps": 1e-5}, "embedding": {"scale": 2.0}, "logit_scale": 0.5,
+         "logit_softcap": 9.0, "residual_mult": 0.8, "layers": layers}
+    c.update(extra)
+    return c
+
+
+@built
+def test_gavodra_configs_are_refused_by_name(tmp_path):
+    serving = load_pkg("serving")
+    att = {"type": "attention", "mlp": None, "mixer": GAVODRA_MIXER}
+
+    def mixer(**kw):
+        return dict(att, mixer=dict(GAVODRA_MIXER, **kw))
+    cases = [(_gavodra_cfg([{"type": "helix", "mixer": {}, "mlp": None}]), "helix"),
+             (_gavodra_cfg([dict(att, mlp={"kind": "sparse"})]), "sparse"),
+             (_gavodra_cfg([dict(att, mlp={"kind": "dense", "ff": 5})]), "limit"),
+             (_gavodra_cfg([dict(att, mlp=dict(GAVODRA_MOE, router={"experts": 3, "top": 2}))]), "scale"),
+             (_gavodra_cfg([dict(att, mixer={k: v for k, v in GAVODRA_MIXER.items() if k != "bias_max"})]), "bias_max"),
+             (_gavodra_cfg([mixer(v_mix=1)]), "true or false"),
+             (_gavodra_cfg([att], logit_softcap=0.0), "logit_softcap"),
+             ({k: v for k, v in _gavodra_cfg([att]).items() if k != "residual_mult"}, "residual_mult")]
+    for cfg, word in cases:
+        (tmp_path / "config.json").write_text(json.dumps(cfg))
+        with pytest.raises(serving.ServingError) as e:
+            serving.ServingEngine(str(tmp_path), "float32", 64, 1)
+        assert word in str(e.value), (word, str(e.value))
+
+
+def test_gavodra_tensor_shapes_cover_a_config():
+    serving = load_pkg("serving")
+    layers = [{"type": "attention", "mixer": GAVODRA_MIXER, "mlp": {"kind": "dense", "ff": 12, "limit": 2.0}},
+              {"type": "attention", "mixer": dict(GAVODRA_MIXER, v_mix=False), "mlp": None},
+              {"type": "attention", "mixer": GAVODRA_MIXER, "mlp": GAVODRA_MOE}]
+    cfg = _gavodra_cfg(layers)
+    t = serving.random_gavodra_tensors(cfg, 0, rel_rows=10)
+    assert t["l0.mix.q"].shape == (24, 16) and t["l0.mix.v"].shape == (10, 16) and t["l0.mix.o"].shape == (16, 20) and t["l0.mix.rel"].shape == (10, 4)
+    assert t["l0.mix.vmix"].shape == () and "l1.mix.vmix" not in t and "l1.norm2" not in t and "head" not in t
+    assert t["l2.mlp.e2.down"].shape == (16, 7) and t["l2.mlp.correction"].shape == (3,) and t["l2.mlp.shared.sg"].shape == (1, 16)
+    assert {k: v.shape for k, v in t.items()} == G.tensor_shapes(cfg, 10)
+
+
+def test_plain_gavodra_statements_agree():
+    assert G.self_check()
+
+
+def test_plain_gavodra_buckets_mixing_and_choice():
+    # 8 rows that end at distance 64: 4 rows of one distance, then factors of 2
+    assert [G.bucket(n, 8, 64) for n in (0, 3, 4, 7, 8, 15, 16, 31, 32, 63, 64, 900)] == [0, 3, 4, 4, 5, 5, 6, 6, 7, 7, 7, 7]
+    assert [G.bucket(n, 2, 5) for n in (0, 1, 7)] == [0, 1, 1]
+    # where the logarithm is not on a step the plain formula says the same
+    for rows, far in ((12, 35), (32, 190), (9, 50)):
+        half = rows // 2
+        for n in range(half, far + 20):
+            v = np.log(n / half) / np.log(far / half) * (rows - half)
+            if abs(v - round(v)) > 1e-9:
+                assert G.bucket(n, rows, far) == min(rows - 1, half + int(np.floor(v)))
+    # the bias reads the key's distance and the query's head
+    tab = np.arange(16.0).reshape(8, 2)
+    b = G.bias_matrix(tab, 64, [9, 10], 11)
+    assert b.shape == (2, 2, 11) and b[1, 0, 9] == 1.0 and b[0, 0, 7] == 4.0 and b[0, 1, 2] == tab[5, 0] and b[0, 0, 0] == tab[5, 0]
+    assert np.allclose(G.mix_values(np.array([2.0, 4.0]), 0.25, np.array([10.0, 0.0])), [4.0, 3.0])
+    # the correction moves the choice, the weights are the plain scores times the factor
+    e, w = G.route(np.array([0.0, 1.0, -1.0]), np.array([0.0, -0.9, 0.3]), 2, 2.0)
+    assert list(e) == [2, 0] and np.allclose(w, 2.0 * G.sigmoid(np.array([-1.0, 0.0])))
+    # the gate is bounded above only, the up value on both sides
+    W = {"gate": np.eye(1), "up": np.eye(1), "down": np.eye(1)}
+    for x in (-3.0, 0.5, 3.0):
+        g, u = min(x, 1.0), min(max(x, -1.0), 1.0)
+        assert np.isclose(G.clamped_glu(np.array([[x]]), W, "", 1.0)[0, 0], g / (1 + np.exp(-1.702 * g)) * (u + 1))
