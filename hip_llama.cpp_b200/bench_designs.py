@@ -5,7 +5,9 @@ design the framework has: latent attention + a recurrent mixer + a looped segmen
 --design bozovik); or of Mozetar beside Numizen -- the closest design the framework has: softmax attention + a gated linear
 recurrence + a mixture of experts behind a softmax router with groups -- and llama2 at equal size (bench.py --design mozetar);
 or of Logulix beside Bozovik (sequential blocks, windowed attention, a recurrent mixer, ungated dense feed-forwards, a looped segment),
-Numizen with dense feed-forwards (the scan its memories share) and llama2 at equal size (bench.py --design logulix).
+Numizen with dense feed-forwards (the scan its memories share) and llama2 at equal size (bench.py --design logulix); or of Gavodra
+beside Mozetar -- the closest design the framework has: softmax attention layers with gated experts behind a corrected router -- and
+Timerax (clamped experts with a shared one) and llama2 at equal size (bench.py --design gavodra).
 
 Random weights at sizes that resemble a real model's layers; a few layers only, so that building the folder stays
 short.  For every size: prompt ingestion (one prompt in one step) and batched decoding (one token per live request per
@@ -142,6 +144,18 @@ def logulix_config(s: dict, n: dict) -> dict:
             "embedding": {"scale": 1.0}, "logit_scale": 0.5, "loop": {"start": 1, "stop": min(3, s["layers"]), "times": 1}}
 
 
+# Gavodra at the same widths, expert sizes and vocabulary: causal attention with heads of 128, bias tables of 32 rows that end at 2048
+# positions, value mixing in every layer; layer 0 has a dense feed-forward as wide as the experts a token uses, the others the mixture.
+def gavodra_config(s: dict, bias_max: int = 2048) -> dict:
+    att = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5, "bias_max": bias_max, "v_mix": True}
+    moe = {"kind": "moe", "expert": {"ff": s["ff"], "limit": 7.0}, "router": {"experts": s["experts"], "top": s["top"], "scale": 2.0},
+           "shared": {"ff": s["sff"], "limit": 7.0}}
+    dense = {"kind": "dense", "ff": s["top"] * s["ff"] + s["sff"], "limit": 7.0}
+    layers = [{"type": "attention", "mixer": att, "mlp": dense if i == 0 else moe} for i in range(s["layers"])]
+    return {"architecture": "Gavodra", "layers": layers, "norm": {"eps": 1e-6}, "vocab": s["vocab"], "width": s["width"], "embedding": {"scale": s["width"] ** 0.5},
+            "residual_mult": 0.8, "logit_scale": 1.0, "logit_softcap": 30.0}
+
+
 def _time_timerax(serving, folder, prompt_len, batch, ctx, steps, warmup, kernels):
     rng = np.random.default_rng(0)
     out = {}
@@ -273,16 +287,34 @@ def run(load_pkg, sizes, prompt_len=4096, batch=64, ctx=512, steps=16, warmup=3,
     for name in sizes:
         s = SIZES[name]
         r = {}
+
+        def arm(cfg, tensors, shapes):
+            tmp = tempfile.mkdtemp(prefix="design_bench_")
+            try:
+                serving.save_model_folder(tmp, cfg, tensors)
+                out = _time_folder(serving, tmp, prompt_len, batch, ctx, steps, warmup, kernels)
+                out["weights_bytes"] = timerax_weight_bytes(cfg, shapes)
+                return out
+            finally:
+                shutil.rmtree(tmp, ignore_errors=True)
+
+        if design == "gavodra":
+            c = gavodra_config(s)
+            if kernels:
+                print(f"# gavodra, {name}", flush=True)
+            r["gavodra"] = arm(c, serving.random_gavodra_tensors(c, 0), serving.gavodra_tensor_shapes(c))
+            c = mozetar_config(s, MOZETAR[name])
+            if kernels:
+                print(f"# mozetar, {name}", flush=True)
+            r["mozetar"] = arm(c, serving.random_mozetar_tensors(c, 0), serving.mozetar_tensor_shapes(c))
+            if not kernels:
+                c = timerax_config(s)
+                r["timerax"] = arm(c, serving.random_timerax_tensors(c, 0), serving.timerax_tensor_shapes(c))
+            if llama:
+                r["llama2_bf16_equal_size"] = _time_llama(engine_mod, checkpoint_mod, s, prompt_len, batch, ctx, steps, warmup)
+            results[name] = r
+            continue
         if design == "logulix":
-            def arm(cfg, tensors, shapes):
-                tmp = tempfile.mkdtemp(prefix="design_bench_")
-                try:
-                    serving.save_model_folder(tmp, cfg, tensors)
-                    out = _time_folder(serving, tmp, prompt_len, batch, ctx, steps, warmup, kernels)
-                    out["weights_bytes"] = timerax_weight_bytes(cfg, shapes)
-                    return out
-                finally:
-                    shutil.rmtree(tmp, ignore_errors=True)
             c = logulix_config(s, LOGULIX[name])
             r["logulix"] = arm(c, serving.random_logulix_tensors(c, 0, decay_rank=64), serving.logulix_tensor_shapes(c, 64))
             if not kernels or llama:
