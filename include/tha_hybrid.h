@@ -43,7 +43,7 @@ extern "C" {
 #define THA_BLOCK_PARALLEL 0   /* x <- x + mixer(norm1 x) + ff(norm x): mixer and feed-forward read the same x */
 #define THA_BLOCK_SEQUENTIAL 1 /* x <- x + m mixer(norm1 x), then x <- x + m ff(norm2 x), then the per-token side input */
 #define THA_BLOCK_STREAMS 2    /* several residual streams: every sublayer reads a weighted sum of them and writes to all (tha_streams_t) */
-#define THA_BLOCK_POST 3       /* x <- x + m norm1(mixer(x)), x <- x + m norm2(ff(x)): the sublayers read x itself, rms norms weigh what they return */
+#define THA_BLOCK_POST 3       /* x <- x + m norm1(mixer(x)), x <- x + m norm2(ff(x)): no norm ahead of a sublayer, rms norms on the results */
 
 #define THA_NORM_RMS 0     /* x / sqrt(mean(x^2) + eps) * (w_offset + w) */
 #define THA_NORM_DYT 1     /* tanh(alpha * x) * w + b: element-wise, no statistics */
